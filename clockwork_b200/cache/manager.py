@@ -67,7 +67,7 @@ class RequestCache:
     num_computed: int = 0  # positions [0, num_computed) have their keys/values (or state) stored
     shared_prefix_pages: int = 0  # leading pages of group 0 owned through the prefix cache
     state_slot: int | None = None
-    live_from: list[int] = field(default_factory=list)  # per group: first logical block still held
+    live_from: list[int] = field(default_factory=list)  # per group: the blocks before this one (but those of kept first tokens) were given back
     table_epoch: int = 0  # counts changes of existing table entries (a copied page): holders of a copy of the table compare it
     writable_len: int = 0  # positions below this need neither a new page nor a copy: the request owns their pages alone
 
@@ -280,8 +280,8 @@ class CacheManager:
 
     def release_behind_window(self, req: RequestCache, computed: int) -> int:
         """Give back pages of windowed groups that no later token can read: a query at position
-        p >= computed reads keys in [p + 1 - window, p] only; in a group whose layers read blocks of positions,
-        keys from the start of p's own block on.  Returns the number given back."""
+        p >= computed reads keys in [p + 1 - window, p] only (and the first ``keep_first`` ones, whose pages stay); in a
+        group whose layers read blocks of positions, keys from the start of p's own block on.  Returns the number given back."""
         given = 0
         for g, group in enumerate(self.groups):
             window, block = group.need.window, group.need.block
@@ -294,7 +294,8 @@ class CacheManager:
                 first_needed = max(first_needed, computed - computed % block)
             keep_from = first_needed // self.page_size
             table = req.tables[g]
-            for blk in range(req.live_from[g], min(keep_from, len(table))):
+            kept_pages = -(-group.need.keep_first // self.page_size)
+            for blk in range(max(req.live_from[g], kept_pages), min(keep_from, len(table))):
                 if table[blk] != NO_PAGE:
                     group.allocator.decref(table[blk])
                     table[blk] = NO_PAGE

@@ -57,6 +57,7 @@ class ExecStep:
     layer: int  # index into ModelSpec.layers (whose weights run)
     cache_layer: int | None = None  # cache written/read; None means ``layer``
     write_cache: bool = True  # False: read what ``cache_layer`` already holds for these tokens
+    add_input: bool = False  # the model's input rows (the embedding as it was before the first run) are added to the residual first
 
     def resolved_cache_layer(self) -> int:
         return self.layer if self.cache_layer is None else self.cache_layer
@@ -77,6 +78,7 @@ class ModelSpec:
     eos_token_ids: tuple[int, ...] = ()
     max_position_embeddings: int | None = None
     embedding_scale: float = 1.0  # the embedding rows are multiplied by this (the output head, if tied, is not)
+    logit_scale: float = 1.0  # the output product is multiplied by this, before ``logit_softcap``
     logit_softcap: float | None = None  # logits <- cap * tanh(logits / cap)
     absolute_positions: PartSpec | None = None  # a position part that adds a vector per position to the embedding
     pair_embedding: PartSpec | None = None  # an embedding part that adds a row chosen by (previous token, token)
@@ -109,15 +111,17 @@ def sequential_schedule(num_layers: int) -> list[ExecStep]:
     return [ExecStep(layer=i) for i in range(num_layers)]
 
 
-def looped_schedule(num_layers: int, start: int, stop: int, times: int) -> list[ExecStep]:
+def looped_schedule(num_layers: int, start: int, stop: int, times: int, add_input: bool = False) -> list[ExecStep]:
     """Layers 0 .. start-1 once, layers start .. stop-1 ``times`` times in a row with the same weights, then the rest.
     Every pass keeps a cache or state of its own: the first pass under the layer's own number, pass p > 0 of layer i under
-    ``num_layers + (p - 1) * (stop - start) + (i - start)``."""
+    ``num_layers + (p - 1) * (stop - start) + (i - start)``.  ``add_input``: every pass but the first begins with the
+    model's input rows added to the residual."""
     if not 0 <= start <= stop <= num_layers or times < 1:
         raise ValueError(f"a loop over layers {start} .. {stop - 1}, {times} times, does not fit {num_layers} layers")
     steps = [ExecStep(layer=i) for i in range(start)]
     for p in range(times):
         for i in range(start, stop):
-            steps.append(ExecStep(layer=i, cache_layer=i if p == 0 else num_layers + (p - 1) * (stop - start) + (i - start)))
+            steps.append(ExecStep(layer=i, cache_layer=i if p == 0 else num_layers + (p - 1) * (stop - start) + (i - start),
+                                  add_input=add_input and p > 0 and i == start))
     steps.extend(ExecStep(layer=i) for i in range(stop, num_layers))
     return steps

@@ -1,4 +1,5 @@
-// Embedding gather and fused residual-add + RMSNorm.
+// Embedding gather and fused residual-add + norm (RMSNorm, or with CENTER layer norm: the row's mean is taken off and
+// the mean of the squared deviations stands in the mean square's place).
 //
 // Reference formulas: clockwork/engine/model.py:200 (embedding), :44-49 (RMSNorm: float32
 // statistics, x * rsqrt(mean(x^2) + eps), then the weight), :150 and :154 (residual sums).
@@ -36,8 +37,8 @@ extern "C" int cw_embed(float* out, const void* table, const int* ids, int N, in
 }
 
 // resid[row] (+= delta[row]); out[r] = weight * (x * rsqrt(mean(x^2)+eps)).
-// With `rows` given, output row r is computed from residual row rows[r] (no add is done).
-template <typename T>
+// With `rows` given, output row r is computed from residual row rows[r] (no add is done).  CENTER: x - mean(x) in x's place.
+template <typename T, bool CENTER>
 __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const T* __restrict__ delta,
                                    const float* __restrict__ weight, T* __restrict__ out,
                                    const int* __restrict__ rows, int num_resid_rows, float eps,
@@ -57,19 +58,28 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const T* __restric
     }
     float* x = resid + (size_t)src_row * H;
     const T* d = delta ? delta + (size_t)src_row * H : nullptr;
-    float ss = 0.f;
+    float ss = 0.f, total = 0.f;
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
         float v = x[c];
         if (d) {
             v += to_f(d[c]);
             x[c] = v;
         }
-        ss = fmaf(v, v, ss);
+        if (CENTER) total += v;
+        else ss = fmaf(v, v, ss);
+    }
+    float mean = 0.f;
+    if (CENTER) {  // the deviations from the mean, in a second pass over the thread's own columns
+        mean = block_sum(total, scratch) / (float)H;
+        for (int c = threadIdx.x; c < H; c += blockDim.x) {
+            const float v = x[c] - mean;
+            ss = fmaf(v, v, ss);
+        }
     }
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)H + eps);
     T* o = out + (size_t)r * H;
-    for (int c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_f<T>(weight[c] * (x[c] * inv));
+    for (int c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_f<T>(weight[c] * ((CENTER ? x[c] - mean : x[c]) * inv));
 }
 
 // The same for many rows (prompt portions): one warp per row, the row held in registers between the
@@ -98,7 +108,33 @@ struct Vec4<bf16> {
     }
 };
 
-template <typename T, int NV>
+// A row held in a warp's registers as v[i] = columns (i*32 + lane)*4 ..: takes the mean off every column that exists.
+template <int NV>
+__device__ __forceinline__ void warp_center(float4 (&v)[NV], int lane, int H) {
+    float total = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+        if ((i * 32 + lane) * 4 < H) total += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    const float mean = warp_sum(total) / (float)H;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
+    }
+}
+
+template <int NV>
+__device__ __forceinline__ float warp_square_sum(const float4 (&v)[NV], int lane, int H) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+        if ((i * 32 + lane) * 4 < H) {
+            ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss);
+            ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
+        }
+    return warp_sum(ss);
+}
+
+template <typename T, int NV, bool CENTER>
 __global__ void __launch_bounds__(256)
 add_rmsnorm_warp_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ weight,
                         T* __restrict__ out, int num_rows, float eps, int H) {
@@ -110,7 +146,6 @@ add_rmsnorm_warp_kernel(float* __restrict__ resid, const T* __restrict__ delta, 
     float* x = resid + (size_t)r * H;
     const T* d = delta ? delta + (size_t)r * H : nullptr;
     float4 v[NV];
-    float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int c = (i * 32 + lane) * 4;
@@ -121,11 +156,10 @@ add_rmsnorm_warp_kernel(float* __restrict__ resid, const T* __restrict__ delta, 
                 v[i].x += dv.x; v[i].y += dv.y; v[i].z += dv.z; v[i].w += dv.w;
                 Vec4<float>::store(x + c, v[i]);
             }
-            ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss);
-            ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
         }
     }
-    ss = warp_sum(ss);
+    if (CENTER) warp_center<NV>(v, lane, H);
+    const float ss = warp_square_sum<NV>(v, lane, H);
     const float inv = 1.0f / sqrtf(ss / (float)H + eps);
     T* o = out + (size_t)r * H;
 #pragma unroll
@@ -138,49 +172,56 @@ add_rmsnorm_warp_kernel(float* __restrict__ resid, const T* __restrict__ delta, 
     }
 }
 
-template <typename T>
+template <typename T, bool CENTER>
 static int launch_rmsnorm_warp(float* resid, const T* delta, const float* weight, T* out, int rows, int H, float eps,
                                cudaStream_t stream) {
     const int warps = 8;
     const dim3 grid((rows + warps - 1) / warps), block(warps * 32);
     const int nv = (H + 127) / 128;
 #define CW_NV(n) \
-    if (nv <= n) return cw_launch(add_rmsnorm_warp_kernel<T, n>, grid, block, 0, stream, 1, resid, delta, weight, out, rows, eps, H);
+    if (nv <= n) return cw_launch(add_rmsnorm_warp_kernel<T, n, CENTER>, grid, block, 0, stream, 1, resid, delta, weight, out, rows, eps, H);
     CW_NV(4) CW_NV(8) CW_NV(12) CW_NV(16) CW_NV(24) CW_NV(32)
 #undef CW_NV
     return CW_ERR_UNSUPPORTED;
 }
 
-extern "C" int cw_add_rmsnorm(float* resid, const void* delta, const float* weight, void* out,
-                              const int* rows, int num_out_rows, int num_resid_rows, int H,
-                              float eps, int dtype, int* status, cudaStream_t stream) {
-    if (num_out_rows == 0) return CW_OK;
-    if (num_out_rows < 0 || H <= 0) return CW_ERR_BAD_SIZE;
-    if (rows != nullptr && delta != nullptr) return CW_ERR_UNSUPPORTED;
+template <typename T, bool CENTER>
+static int launch_add_rmsnorm(float* resid, const T* delta, const float* weight, T* out, const int* rows, int num_out_rows,
+                              int num_resid_rows, int H, float eps, int* status, cudaStream_t stream) {
     // many rows: a warp per row; few rows (decode): a block per row, for the latency of the one row
     const bool aligned = H % 4 == 0 && H <= 4096 && ((uintptr_t)resid & 15) == 0 && ((uintptr_t)weight & 15) == 0 &&
                          ((uintptr_t)out & 15) == 0 && ((uintptr_t)delta & 15) == 0;
-    if (rows == nullptr && num_out_rows >= 256 && aligned) {
-        if (dtype == 0)
-            return launch_rmsnorm_warp<float>(resid, (const float*)delta, weight, (float*)out, num_out_rows, H, eps, stream);
-        if (dtype == 1)
-            return launch_rmsnorm_warp<bf16>(resid, (const bf16*)delta, weight, (bf16*)out, num_out_rows, H, eps, stream);
-        return CW_ERR_BAD_DTYPE;
-    }
+    if (rows == nullptr && num_out_rows >= 256 && aligned)
+        return launch_rmsnorm_warp<T, CENTER>(resid, delta, weight, out, num_out_rows, H, eps, stream);
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
+    return cw_launch(add_rmsnorm_kernel<T, CENTER>, dim3(num_out_rows), dim3(threads), 0, stream, 1, resid, delta, weight, out, rows,
+                     num_resid_rows, eps, H, status);
+}
+
+// center: 0 RMSNorm, 1 layer norm
+extern "C" int cw_add_rmsnorm(float* resid, const void* delta, const float* weight, void* out,
+                              const int* rows, int num_out_rows, int num_resid_rows, int H,
+                              float eps, int center, int dtype, int* status, cudaStream_t stream) {
+    if (num_out_rows == 0) return CW_OK;
+    if (num_out_rows < 0 || H <= 0) return CW_ERR_BAD_SIZE;
+    if (rows != nullptr && delta != nullptr) return CW_ERR_UNSUPPORTED;
     if (dtype == 0)
-        return cw_launch(add_rmsnorm_kernel<float>, dim3(num_out_rows), dim3(threads), 0, stream, 1, resid,
-                         (const float*)delta, weight, (float*)out, rows, num_resid_rows, eps, H, status);
+        return center ? launch_add_rmsnorm<float, true>(resid, (const float*)delta, weight, (float*)out, rows, num_out_rows, num_resid_rows, H,
+                                                        eps, status, stream)
+                      : launch_add_rmsnorm<float, false>(resid, (const float*)delta, weight, (float*)out, rows, num_out_rows, num_resid_rows, H,
+                                                         eps, status, stream);
     if (dtype == 1)
-        return cw_launch(add_rmsnorm_kernel<bf16>, dim3(num_out_rows), dim3(threads), 0, stream, 1, resid,
-                         (const bf16*)delta, weight, (bf16*)out, rows, num_resid_rows, eps, H, status);
+        return center ? launch_add_rmsnorm<bf16, true>(resid, (const bf16*)delta, weight, (bf16*)out, rows, num_out_rows, num_resid_rows, H,
+                                                       eps, status, stream)
+                      : launch_add_rmsnorm<bf16, false>(resid, (const bf16*)delta, weight, (bf16*)out, rows, num_out_rows, num_resid_rows, H,
+                                                        eps, status, stream);
     return CW_ERR_BAD_DTYPE;
 }
 
 // resid[r] += parts[0][r] + parts[1][r] + .. (in this order: the splits of a product over K that were
 // kept apart), then, with `out`, out[r] = resid[r] normalised as above.  A warp per row, the row in
-// registers between the two passes.
-template <typename T, int NV>
+// registers between the two passes.  CENTER as above.
+template <typename T, int NV, bool CENTER>
 __global__ void __launch_bounds__(256)
 add_parts_rmsnorm_kernel(float* __restrict__ resid, const float* __restrict__ parts, int num_parts, size_t part_stride,
                          const float* __restrict__ weight, T* __restrict__ out, int num_rows, float eps, int H) {
@@ -191,7 +232,6 @@ add_parts_rmsnorm_kernel(float* __restrict__ resid, const float* __restrict__ pa
     if (r >= num_rows) return;
     float* x = resid + (size_t)r * H;
     float4 v[NV];
-    float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int c = (i * 32 + lane) * 4;
@@ -211,14 +251,11 @@ add_parts_rmsnorm_kernel(float* __restrict__ resid, const float* __restrict__ pa
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
         const int c = (i * 32 + lane) * 4;
-        if (c < H) {
-            Vec4<float>::store(x + c, v[i]);
-            ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss);
-            ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
-        }
+        if (c < H) Vec4<float>::store(x + c, v[i]);
     }
     if (out == nullptr) return;
-    ss = warp_sum(ss);
+    if (CENTER) warp_center<NV>(v, lane, H);
+    const float ss = warp_square_sum<NV>(v, lane, H);
     const float inv = 1.0f / sqrtf(ss / (float)H + eps);
     T* o = out + (size_t)r * H;
 #pragma unroll
@@ -231,14 +268,14 @@ add_parts_rmsnorm_kernel(float* __restrict__ resid, const float* __restrict__ pa
     }
 }
 
-template <typename T>
+template <typename T, bool CENTER>
 static int launch_add_parts(float* resid, const float* parts, int num_parts, size_t part_stride, const float* weight, T* out,
                             int rows, int H, float eps, cudaStream_t stream) {
     const int warps = 8;
     const dim3 grid((rows + warps - 1) / warps), block(warps * 32);
     const int nv = (H + 127) / 128;
 #define CW_NV(n) \
-    if (nv <= n) return cw_launch(add_parts_rmsnorm_kernel<T, n>, grid, block, 0, stream, 1, resid, parts, num_parts, part_stride, weight, out, rows, eps, H);
+    if (nv <= n) return cw_launch(add_parts_rmsnorm_kernel<T, n, CENTER>, grid, block, 0, stream, 1, resid, parts, num_parts, part_stride, weight, out, rows, eps, H);
     CW_NV(4) CW_NV(8) CW_NV(12) CW_NV(16) CW_NV(24) CW_NV(32)
 #undef CW_NV
     return CW_ERR_UNSUPPORTED;
@@ -247,16 +284,19 @@ static int launch_add_parts(float* resid, const float* parts, int num_parts, siz
 // parts: float32 [num_parts][part_rows][H] (part_rows >= rows); out null: only the sum.  H a multiple of 4,
 // at most 4096; 16-byte aligned pointers; CW_ERR_UNSUPPORTED otherwise.
 extern "C" int cw_add_parts_rmsnorm(float* resid, const float* parts, int num_parts, int part_rows, const float* weight,
-                                    void* out, int rows, int H, float eps, int dtype, cudaStream_t stream) {
+                                    void* out, int rows, int H, float eps, int center, int dtype, cudaStream_t stream) {
     if (rows == 0) return CW_OK;
     if (rows < 0 || H <= 0 || num_parts < 1 || part_rows < rows) return CW_ERR_BAD_SIZE;
     if (H % 4 != 0 || H > 4096 || ((uintptr_t)resid & 15) || ((uintptr_t)parts & 15) || ((uintptr_t)weight & 15) ||
         ((uintptr_t)out & 15))
         return CW_ERR_UNSUPPORTED;
     const size_t stride = (size_t)part_rows * H;
-    if (out == nullptr || dtype == 0)
-        return launch_add_parts<float>(resid, parts, num_parts, stride, weight, (float*)out, rows, H, eps, stream);
-    if (dtype == 1) return launch_add_parts<bf16>(resid, parts, num_parts, stride, weight, (bf16*)out, rows, H, eps, stream);
+    if (out == nullptr || (dtype == 0 && !center))
+        return launch_add_parts<float, false>(resid, parts, num_parts, stride, weight, (float*)out, rows, H, eps, stream);
+    if (dtype == 0) return launch_add_parts<float, true>(resid, parts, num_parts, stride, weight, (float*)out, rows, H, eps, stream);
+    if (dtype == 1)
+        return center ? launch_add_parts<bf16, true>(resid, parts, num_parts, stride, weight, (bf16*)out, rows, H, eps, stream)
+                      : launch_add_parts<bf16, false>(resid, parts, num_parts, stride, weight, (bf16*)out, rows, H, eps, stream);
     return CW_ERR_BAD_DTYPE;
 }
 
@@ -393,19 +433,21 @@ extern "C" int cw_sum_rmsnorm_add(float* resid, const float* a, const float* b, 
     return cw_launch_ordered(sum_rmsnorm_add_kernel, dim3(N), dim3(threads), 0, stream, resid, a, b, ca, cb, w, eps, W);
 }
 
-// ---- logits bent towards a bound ------------------------------------------------------------------------
-// x <- cap tanh(x / cap), in place, float32.
-__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long n, float cap) {
+// ---- logits scaled and bent towards a bound ---------------------------------------------------------------
+// x <- cap tanh(scale x / cap), in place, float32 (cap 0: x <- scale x).
+__global__ void __launch_bounds__(256) softcap_kernel(float* __restrict__ x, long long n, float cap, float scale) {
     pdl_wait();
-    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x)
-        x[i] = cap * tanhf(x[i] / cap);
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (long long)gridDim.x * blockDim.x) {
+        const float z = x[i] * scale;  // (scale 1: the logit as it is)
+        x[i] = cap > 0.f ? cap * tanhf(z / cap) : z;
+    }
 }
 
-extern "C" int cw_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+extern "C" int cw_softcap(float* x, long long n, float cap, float scale, cudaStream_t stream) {
     if (n == 0) return CW_OK;
-    if (n < 0 || !(cap > 0.f)) return CW_ERR_BAD_SIZE;
+    if (n < 0 || !(cap >= 0.f)) return CW_ERR_BAD_SIZE;
     const int blocks = (int)min((long long)148 * 8, (n + 255) / 256);
-    return cw_launch_ordered(softcap_kernel, dim3(blocks), dim3(256), 0, stream, x, n, cap);
+    return cw_launch_ordered(softcap_kernel, dim3(blocks), dim3(256), 0, stream, x, n, cap, scale);
 }
 
 // ---- a second table read by a hash of (previous token, token) -------------------------------------------

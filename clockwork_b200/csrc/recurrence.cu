@@ -14,11 +14,12 @@
 //                       float32 state, one pass over the portion in token order
 //   cw_gated_group_norm y (*silu(z)) divided by its root mean square in equal parts, times a weight
 //                       (times silu(z)): the gate before or after the norm
+//   cw_rotate_heads     the leading entries of every head of a row turned by the token's position (rotation.cuh), in place
 //   cw_activation       gelu (tanh form), tanh, silu, sigmoid, in place (cw_activation_cols: on some columns of wider rows)
 //
 // Everything that enters the recurrence (decays, step sizes, the state, the norm) is float32 in both
 // run precisions; T only names the type of activations that matrix products read or wrote.
-#include "common.cuh"
+#include "rotation.cuh"
 
 // ---- token shift ----------------------------------------------------------------------------------
 template <typename T>
@@ -464,8 +465,8 @@ extern "C" int cw_bounded_forget(float* x, int ld, const float* bias, const floa
 // ---- gated norm in parts ----------------------------------------------------------------------------
 // y [N, C] float32, gate z [N, ldz] float32.  mode bit 0 (gate first): u = y gate(z), out = u / rms_part(u) * weight.
 // Otherwise: out = y / rms_part(y) * weight * gate(z).  mode bit 1: gate = sigmoid (else silu).  mode bit 2: every
-// part uses the same weight of one part's width.  mode bit 3: no gate at all (z may be null).  A block per (row, part);
-// sums in a fixed order.
+// part uses the same weight of one part's width.  mode bit 3: no gate at all (z may be null).  weight null: none is
+// multiplied.  A block per (row, part); sums in a fixed order.
 template <typename T>
 __global__ void __launch_bounds__(256)
 gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z, int ldz, const float* __restrict__ weight,
@@ -479,7 +480,7 @@ gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z
     const int width = C / parts;
     const float* yr = y + (size_t)row * C + (size_t)p * width;
     const float* zr = z + (size_t)row * ldz + (size_t)p * width;
-    const float* wr = weight + ((mode & 4) ? 0 : (size_t)p * width);
+    const float* wr = weight != nullptr ? weight + ((mode & 4) ? 0 : (size_t)p * width) : nullptr;
     float ss = 0.f;
     for (int c = threadIdx.x; c < width; c += blockDim.x) {
         float u = yr[c];
@@ -495,7 +496,7 @@ gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z
         const float g = ungated ? 0.f : zr[c];
         const float sg = ungated ? 1.f : (plain_sigmoid ? 1.f : g) / (1.f + expf(-g));
         const float u = gate_first ? yr[c] * sg : yr[c];
-        float r = u * inv * wr[c];
+        float r = wr != nullptr ? u * inv * wr[c] : u * inv;
         if (!gate_first) r *= sg;
         out[(size_t)row * C + (size_t)p * width + c] = from_f<T>(r);
     }
@@ -517,6 +518,41 @@ extern "C" int cw_gated_group_norm(const float* y, const float* z, int ldz, cons
         return cw_launch_ordered(gated_group_norm_kernel<bf16>, grid, dim3(threads), 0, stream, y, z, ldz, weight, (bf16*)out, C, parts,
                          eps, mode);
     return CW_ERR_BAD_DTYPE;
+}
+
+// ---- rotary positions in place ---------------------------------------------------------------------------
+// x [N, ld] float32: `heads` heads of dk columns, the leading rot.dims entries of each turned by positions[n].  A block per
+// token: the pairs' sines and cosines once, then a thread per pair of entries.
+__global__ void __launch_bounds__(256)
+rotate_heads_kernel(float* __restrict__ x, int ld, const int* __restrict__ positions, Rotation rot, int heads, int dk) {
+    extern __shared__ float rh_table[];
+    pdl_wait();
+    const int n = blockIdx.x, half = rot.dims >> 1;
+    float* cs = rh_table;
+    float* sn = rh_table + half;
+    rotation_table(rot, positions[n], cs, sn);
+    __syncthreads();
+    float* row = x + (size_t)n * ld;
+    for (int c = threadIdx.x; c < heads * half; c += blockDim.x) {
+        const int h = c / half, i = c - h * half;
+        float* head = row + (size_t)h * dk;
+        const int first = rotation_first(rot, i), second = rotation_second(rot, i);
+        const float u = head[first], v = head[second];
+        head[first] = u * cs[i] - v * sn[i];
+        head[second] = v * cs[i] + u * sn[i];
+    }
+}
+
+extern "C" int cw_rotate_heads(float* x, int ld, const int* positions, const float* inv_freq, int rot_dims, int interleaved,
+                               float amplitude, int N, int heads, int dk, cudaStream_t stream) {
+    if (N == 0 || rot_dims == 0) return CW_OK;
+    const Rotation rot = {inv_freq, rot_dims, interleaved, amplitude};
+    if (N < 0 || heads <= 0 || dk <= 0 || !rotation_ok(rot, dk) || ld < heads * dk || positions == nullptr) return CW_ERR_BAD_SIZE;
+    if (rot_dims > 8192) return CW_ERR_UNSUPPORTED;
+    int threads = 64;
+    while (threads < 256 && threads < heads * (rot_dims >> 1)) threads *= 2;
+    return cw_launch_ordered(rotate_heads_kernel, dim3(N), dim3(threads), sizeof(float) * (size_t)rot_dims, stream, x, ld, positions, rot,
+                             heads, dk);
 }
 
 // ---- activations in place -----------------------------------------------------------------------------

@@ -5,8 +5,11 @@
 //   cw_unit_heads          every head of a row divided by sqrt(sum of squares + eps), times a scale (one scale for the
 //                          leading heads, another for the rest), in place
 //   cw_delta_coefficients  a[t, h, i] = exp(-exp(A[h]) softplus(pre[t, h, i] + dt[h, i])) and beta[t, h] = sigmoid(.), in place
-//   cw_delta_scan          the gated delta rule with a decay per key channel:
+//   cw_delta_prepare       everything between a delta layer's joint product and its scan in one kernel: short convolutions and
+//                          SiLU on q, k, v, unit vectors per q and k head, one decay and one write strength per head
+//   cw_delta_scan          the gated delta rule with a decay per key channel, or one per head:
 //                              S <- diag(a_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  y_t = S^T q_t
+//                          and, if asked, the convolutions' last inputs kept for the next step
 //   cw_gate_scan           the scalar part of a matrix memory with exponential gates, per request and head in token order:
 //                              li = cap tanh((zi + bi)/cap), lf = log sigmoid(cap tanh((zf + bf)/cap)),
 //                              m_t = max(lf + m_(t-1), li);  keep = exp(lf + m_(t-1) - m_t), take = exp(li - m_t), floor = exp(-m_t)
@@ -72,13 +75,96 @@ extern "C" int cw_delta_coefficients(float* pre, int ldp, const float* dt_bias, 
     return cw_launch_ordered(delta_coefficients_kernel, dim3(blocks), dim3(256), 0, stream, pre, ldp, dt_bias, a_log, beta, ldb, N, H, Dk);
 }
 
+// ---- from the joint product to the scan's operands ----------------------------------------------------------
+// x [N, ldx] float32: a token's product row [q (groups*dk) | k (groups*dk) | v (H*dv) | ..], C = 2*groups*dk + H*dv columns
+// that pass a causal convolution of `taps` taps per channel (weight [C, taps], the current token's last; inputs before a
+// portion's first row are the rows kept in the request's state) and SiLU; then every q and k head is divided by
+// sqrt(sum of squares + eps), q heads times q_scale.  out [N, C].  beta [N, ldb] and decay [N, lda] hold the pre-activations of a
+// number per head: coef [N, 2H] = [exp(-exp(A[h]) softplus(decay + dt[h])) | sigmoid(beta)].  A block per token; a warp per q or
+// k head, its channels in registers between the sum and the division.
+#define DP_CH 8  // channels of a head per lane (heads up to 256 wide)
+__global__ void __launch_bounds__(256)
+delta_prepare_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ weight, int taps,
+                     const float* __restrict__ state, long long state_stride, long long conv_off, const long long* __restrict__ slots,
+                     const int* __restrict__ tok_seq, const int* __restrict__ q_start, int groups, int Dk, int H, int Dv, float eps,
+                     float q_scale, const float* __restrict__ beta, int ldb, const float* __restrict__ decay, int lda,
+                     const float* __restrict__ dt_bias, const float* __restrict__ a_log, float* __restrict__ out,
+                     float* __restrict__ coef) {
+    pdl_wait();
+    const int row = blockIdx.x, tid = threadIdx.x;
+    const int qk = groups * Dk, C = 2 * qk + H * Dv, R = taps - 1;
+    float* o = out + (size_t)row * C;
+    float* cf = coef + (size_t)row * 2 * H;
+    const int seq = tok_seq[row];
+    if (seq < 0) {  // padding of a fixed-shape step
+        for (int c = tid; c < C; c += blockDim.x) o[c] = 0.f;
+        for (int h = tid; h < 2 * H; h += blockDim.x) cf[h] = 0.f;
+        return;
+    }
+    const int start = q_start[seq];
+    const float* kept = state + slots[seq] * state_stride + conv_off;
+    auto conv = [&](int c) {
+        float acc = 0.f;
+        for (int j = 0; j < taps; ++j) {
+            const int src = row - (R - j);
+            const float v = src >= start ? x[(size_t)src * ldx + c] : kept[(size_t)(R - (start - src)) * C + c];
+            acc = fmaf(weight[(size_t)c * taps + j], v, acc);
+        }
+        return acc / (1.f + expf(-acc));
+    };
+    const int warp = tid >> 5, lane = tid & 31, nwarps = blockDim.x >> 5;
+    for (int head = warp; head < 2 * groups; head += nwarps) {
+        float u[DP_CH], ss = 0.f;
+#pragma unroll
+        for (int r = 0; r < DP_CH; ++r) {
+            const int i = lane + 32 * r;
+            u[r] = i < Dk ? conv(head * Dk + i) : 0.f;
+            ss = fmaf(u[r], u[r], ss);
+        }
+        ss = warp_sum(ss);
+        const float f = (head < groups ? q_scale : 1.f) / sqrtf(ss + eps);
+#pragma unroll
+        for (int r = 0; r < DP_CH; ++r) {
+            const int i = lane + 32 * r;
+            if (i < Dk) o[head * Dk + i] = u[r] * f;
+        }
+    }
+    for (int c = 2 * qk + tid; c < C; c += blockDim.x) o[c] = conv(c);
+    for (int h = tid; h < H; h += blockDim.x) {
+        const float z = decay[(size_t)row * lda + h] + dt_bias[h];
+        const float step = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+        cf[h] = expf(-expf(a_log[h]) * step);
+        cf[H + h] = 1.f / (1.f + expf(-beta[(size_t)row * ldb + h]));
+    }
+}
+
+extern "C" int cw_delta_prepare(const float* x, int ldx, const float* weight, int taps, const float* state, long long state_stride,
+                                long long conv_off, const long long* slots, const int* tok_seq, const int* q_start, int groups, int Dk,
+                                int H, int Dv, float eps, float q_scale, const float* beta, int ldb, const float* decay, int lda,
+                                const float* dt_bias, const float* a_log, int N, float* out, float* coef, cudaStream_t stream) {
+    if (N == 0) return CW_OK;
+    if (N < 0 || groups <= 0 || Dk <= 0 || H <= 0 || Dv <= 0 || taps <= 0 || ldx < 2 * groups * Dk + H * Dv || ldb < H || lda < H)
+        return CW_ERR_BAD_SIZE;
+    if (Dk > 32 * DP_CH) return CW_ERR_UNSUPPORTED;
+    int threads = 64;
+    while (threads < 256 && threads * 4 < 2 * groups * Dk + H * Dv) threads *= 2;
+    return cw_launch_ordered(delta_prepare_kernel, dim3(N), dim3(threads), 0, stream, x, ldx, weight, taps, state, state_stride, conv_off,
+                             slots, tok_seq, q_start, groups, Dk, H, Dv, eps, q_scale, beta, ldb, decay, lda, dt_bias, a_log, out, coef);
+}
+
 // ---- the delta rule ---------------------------------------------------------------------------------------
 // State per request and head: S [Dk, Dv] stored value-column-major (element (i, j) of head h at (h*Dv + j)*Dk + i).
-// Blocks: (request, head, slice of JB value columns); IP threads share a value column, a thread owns key channels
-// ipart, ipart + IP, ..  The operands of DC tokens at a time are staged in shared memory by cp.async (the next chunk
-// while the current one runs).  Per token the column's S^T k is summed over the IP lanes by shuffles (the update needs
-// it); the read-out sums wait until the chunk is through.  Every sum has a fixed order, so a row's result does not
-// depend on how the request's tokens were cut into steps or on what else the step holds.
+// Blocks: (request, head, slice of JB value columns); IP threads share a value column.  The operands of DC tokens at a time
+// are staged in shared memory by cp.async (the next chunk while the current one runs).  Per token the column's S^T k is
+// summed over the IP lanes by shuffles (the update needs it); the read-out sums wait until the chunk is through.  Every sum
+// has a fixed order, so a row's result does not depend on how the request's tokens were cut into steps or on what else the
+// step holds.
+// IPT > 0: IP known at compile time and heads of whole groups of eight channels at 16-byte addresses: a thread owns channels
+// 4 ipart .. 4 ipart + 3 and the same four in the upper half of the head (two 16-byte words per operand and token), and the
+// read-out sums of the chunk's tokens are added up over the lanes with the tokens spread over them.  IPT = 0: any head size,
+// channels ipart, ipart + IP, .. one word at a time.
+// HEAD: one decay per head and token (a [N, H]) instead of one per key channel (a [N, H*Dk]); S^T k of the decayed state is then
+// the decay times S^T k of the state before.
 #define DS 8    // key channels per thread
 #define DC 16   // tokens per staged chunk
 
@@ -91,72 +177,111 @@ __device__ __forceinline__ void dcp16(float* smem, const float* gmem) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(gmem) : "memory");
 }
 
+struct DeltaScanArgs {
+    const float* q;  // [N, ldq]: head h reads columns (h / heads_per_group) * Dk ..
+    int ldq;
+    const float* k;
+    int ldk;
+    const float* v;  // [N, ldv]: head h's columns h*Dv ..
+    int ldv;
+    const float* a;  // decays
+    int lda;
+    const float* beta;  // [N, ldb]
+    int ldb;
+    float* state;
+    long long state_stride, state_off;
+    const long long* slots;
+    const int* tok_seq;
+    const int* q_start;
+    int Dk, Dv, heads_per_group, IP, wide;
+    float* out;  // [N, ldo]
+    int ldo;
+    // the rows of `carry` [N, ldc] (C columns) that the next step's convolutions read again: the last R of each portion go to
+    // the request's state at carry_off (null: none; the convolutions of this step have run)
+    const float* carry;
+    int ldc, C, R;
+    long long carry_off;
+};
+
+template <int IPT, bool HEAD>
 __global__ void __launch_bounds__(256)
-delta_scan_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk, const float* __restrict__ v, int ldv,
-                  const float* __restrict__ a, int lda, const float* __restrict__ beta, int ldb, float* __restrict__ state,
-                  long long state_stride, long long state_off, const long long* __restrict__ slots, const int* __restrict__ tok_seq,
-                  const int* __restrict__ q_start, int Dk, int Dv, int heads_per_group, int IP, int wide, float* __restrict__ out,
-                  int ldo) {
+delta_scan_kernel(const DeltaScanArgs g) {
     extern __shared__ __align__(16) float ds_smem[];
     pdl_wait();
     const int seq = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
-    const int start = q_start[seq], end = q_start[seq + 1];
+    const int start = g.q_start[seq], end = g.q_start[seq + 1];
     if (end <= start) return;
+    constexpr bool VEC = IPT > 0;
+    const int IP = VEC ? IPT : g.IP, Dk = g.Dk, Dv = g.Dv;
     const int ipart = tid % IP, jl = tid / IP, JB = blockDim.x / IP;
     const int j0 = blockIdx.z * JB, j = j0 + jl;
     const bool live = j < Dv;
-    if (tok_seq[start] < 0) {  // padding rows of a fixed-shape step: no request, no state
+    if (g.tok_seq[start] < 0) {  // padding rows of a fixed-shape step: no request, no state
         if (live && ipart == 0)
-            for (int t = start; t < end; ++t) out[(size_t)t * ldo + (size_t)h * Dv + j] = 0.f;
+            for (int t = start; t < end; ++t) g.out[(size_t)t * g.ldo + (size_t)h * Dv + j] = 0.f;
         return;
     }
-    // one buffer: q [DC][Dk], k [DC][Dk], a [DC][Dk], v [DC][JB], beta [DC]
-    const int buf_words = 3 * DC * Dk + DC * JB + DC;
-    const int g = h / heads_per_group;
-    float* S_mem = state + slots[seq] * state_stride + state_off + ((size_t)h * Dv + (live ? j : 0)) * Dk;
+    // one buffer: q [DC][Dk], k [DC][Dk], a [DC][Dk] or [DC], v [DC][JB], beta [DC]
+    const int a_words = HEAD ? DC : DC * Dk;
+    const int buf_words = 2 * DC * Dk + a_words + DC * JB + DC;
+    const int group = h / g.heads_per_group;
+    float* row_state = g.state + g.slots[seq] * g.state_stride;
+    float* S_mem = row_state + g.state_off + ((size_t)h * Dv + (live ? j : 0)) * Dk;
+    const int half = Dk >> 1;
+    const bool mine = ipart * DS < Dk;  // (VEC: the thread owns channels at all)
+    auto channel = [&](int r) { return VEC ? (r < 4 ? 0 : half) + ipart * 4 + (r & 3) : ipart + r * IP; };
+    auto owns = [&](int r) { return VEC ? mine : ipart + r * IP < Dk; };
     float S[DS];
 #pragma unroll
-    for (int r = 0; r < DS; ++r) {
-        const int i = ipart + r * IP;
-        S[r] = (i < Dk && live) ? S_mem[i] : 0.f;
-    }
-    const float* qp = q + (size_t)g * Dk;
-    const float* kp = k + (size_t)g * Dk;
-    const float* ap = a + (size_t)h * Dk;
-    const float* vp = v + (size_t)h * Dv + j0;
-    const float* bp = beta + h;
+    for (int r = 0; r < DS; ++r) S[r] = (owns(r) && live) ? S_mem[channel(r)] : 0.f;
+    const float* qp = g.q + (size_t)group * Dk;
+    const float* kp = g.k + (size_t)group * Dk;
+    const float* ap = g.a + (HEAD ? (size_t)h : (size_t)h * Dk);
+    const float* vp = g.v + (size_t)h * Dv + j0;
+    const float* bp = g.beta + h;
     const int nv = min(JB, Dv - j0);
     auto fetch = [&](int t0, float* buf) {
         const int n = min(DC, end - t0);
         float* qs = buf;
         float* ks = buf + DC * Dk;
         float* as = buf + 2 * DC * Dk;
-        float* vs = buf + 3 * DC * Dk;
+        float* vs = as + a_words;
         float* bs = vs + DC * JB;
-        if (wide) {  // rows of whole 16-byte pieces at 16-byte addresses
+        if (VEC || g.wide) {  // rows of whole 16-byte pieces at 16-byte addresses
             const int pieces = Dk >> 2;
             for (int idx = tid; idx < n * pieces; idx += blockDim.x) {
                 const int t = idx / pieces, i = (idx - t * pieces) << 2;
-                dcp16(qs + t * Dk + i, qp + (size_t)(t0 + t) * ldq + i);
-                dcp16(ks + t * Dk + i, kp + (size_t)(t0 + t) * ldk + i);
-                dcp16(as + t * Dk + i, ap + (size_t)(t0 + t) * lda + i);
+                dcp16(qs + t * Dk + i, qp + (size_t)(t0 + t) * g.ldq + i);
+                dcp16(ks + t * Dk + i, kp + (size_t)(t0 + t) * g.ldk + i);
+                if (!HEAD) dcp16(as + t * Dk + i, ap + (size_t)(t0 + t) * g.lda + i);
             }
         } else {
             for (int idx = tid; idx < n * Dk; idx += blockDim.x) {
                 const int t = idx / Dk, i = idx - t * Dk;
-                dcp4(qs + idx, qp + (size_t)(t0 + t) * ldq + i);
-                dcp4(ks + idx, kp + (size_t)(t0 + t) * ldk + i);
-                dcp4(as + idx, ap + (size_t)(t0 + t) * lda + i);
+                dcp4(qs + idx, qp + (size_t)(t0 + t) * g.ldq + i);
+                dcp4(ks + idx, kp + (size_t)(t0 + t) * g.ldk + i);
+                if (!HEAD) dcp4(as + idx, ap + (size_t)(t0 + t) * g.lda + i);
             }
         }
         for (int idx = tid; idx < n * nv; idx += blockDim.x) {
             const int t = idx / nv, c = idx - t * nv;
-            dcp4(vs + t * JB + c, vp + (size_t)(t0 + t) * ldv + c);
+            dcp4(vs + t * JB + c, vp + (size_t)(t0 + t) * g.ldv + c);
         }
-        for (int t = tid; t < n; t += blockDim.x) dcp4(bs + t, bp + (size_t)(t0 + t) * ldb);
+        for (int t = tid; t < n; t += blockDim.x) {
+            dcp4(bs + t, bp + (size_t)(t0 + t) * g.ldb);
+            if (HEAD) dcp4(as + t, ap + (size_t)(t0 + t) * g.lda);
+        }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(start, ds_smem);
+    if (g.carry != nullptr) {  // the blocks of the request share its channels out
+        const int n = end - start, block = blockIdx.y * gridDim.z + blockIdx.z, blocks = gridDim.y * gridDim.z;
+        float* kept = row_state + g.carry_off;
+        for (int c = block * blockDim.x + tid; c < g.C; c += blocks * blockDim.x)
+            for (int d = g.R; d >= 1; --d)  // ascending writes; what is read lies ahead of what was written
+                kept[(size_t)(g.R - d) * g.C + c] =
+                    d <= n ? g.carry[(size_t)(end - d) * g.ldc + c] : kept[(size_t)(g.R - (d - n)) * g.C + c];
+    }
     int which = 0;
     for (int t0 = start; t0 < end; t0 += DC, which ^= 1) {
         const int n = min(DC, end - t0);
@@ -164,86 +289,157 @@ delta_scan_kernel(const float* __restrict__ q, int ldq, const float* __restrict_
         const float* qs = buf;
         const float* ks = buf + DC * Dk;
         const float* as = buf + 2 * DC * Dk;
-        const float* vs = buf + 3 * DC * Dk;
+        const float* vs = as + a_words;
         const float* bs = vs + DC * JB;
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // this chunk has landed; everyone has left the other buffer
         if (t0 + DC < end) fetch(t0 + DC, ds_smem + (which ^ 1) * buf_words);
         float part[DC];
+        auto token = [&](int t) {
+            float kc[DS], qc[DS], ac[DS];
+            if (VEC) {
+                const int at = t * Dk + ipart * 4, up = at + half;
+                if (mine) {
+                    *(float4*)&kc[0] = *(const float4*)(ks + at);
+                    *(float4*)&kc[4] = *(const float4*)(ks + up);
+                    *(float4*)&qc[0] = *(const float4*)(qs + at);
+                    *(float4*)&qc[4] = *(const float4*)(qs + up);
+                    if (!HEAD) {
+                        *(float4*)&ac[0] = *(const float4*)(as + at);
+                        *(float4*)&ac[4] = *(const float4*)(as + up);
+                    }
+                } else {
 #pragma unroll
-        for (int t = 0; t < DC; ++t) {
-            part[t] = 0.f;
-            if (t < n) {
-                float kc[DS], aS[DS];
-                float dot0 = 0.f, dot1 = 0.f;  // two chains, added at the end: the same order for every token and batch
+                    for (int r = 0; r < DS; ++r) kc[r] = qc[r] = ac[r] = 0.f;
+                }
+            } else {
 #pragma unroll
                 for (int r = 0; r < DS; ++r) {
                     const int i = ipart + r * IP;
                     const bool on = i < Dk;
                     kc[r] = on ? ks[t * Dk + i] : 0.f;
-                    aS[r] = on ? as[t * Dk + i] * S[r] : 0.f;
-                    if (r & 1) dot1 = fmaf(aS[r], kc[r], dot1);
-                    else dot0 = fmaf(aS[r], kc[r], dot0);
+                    qc[r] = on ? qs[t * Dk + i] : 0.f;
+                    if (!HEAD) ac[r] = on ? as[t * Dk + i] : 0.f;
                 }
-                float dot = dot0 + dot1;
-                for (int o = 1; o < IP; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-                const float u = live ? bs[t] * (vs[t * JB + jl] - dot) : 0.f;
-                float sum0 = 0.f, sum1 = 0.f;
-#pragma unroll
-                for (int r = 0; r < DS; ++r) {
-                    const int i = ipart + r * IP;
-                    S[r] = fmaf(kc[r], u, aS[r]);
-                    const float qc = i < Dk ? qs[t * Dk + i] : 0.f;
-                    if (r & 1) sum1 = fmaf(qc, S[r], sum1);
-                    else sum0 = fmaf(qc, S[r], sum0);
-                }
-                part[t] = sum0 + sum1;
             }
-        }
+            const float decay = HEAD ? as[t] : 0.f;
+            float aS[DS];
+            float dot0 = 0.f, dot1 = 0.f;  // two chains, added at the end: the same order for every token and batch
 #pragma unroll
-        for (int t = 0; t < DC; ++t)
-            for (int o = 1; o < IP; o <<= 1) part[t] += __shfl_xor_sync(0xffffffffu, part[t], o);
-        if (live && ipart == 0) {
+            for (int r = 0; r < DS; ++r) {
+                aS[r] = (HEAD ? decay : ac[r]) * S[r];
+                if (r & 1) dot1 = fmaf(HEAD ? S[r] : aS[r], kc[r], dot1);
+                else dot0 = fmaf(HEAD ? S[r] : aS[r], kc[r], dot0);
+            }
+            float dot = dot0 + dot1;
+            if (VEC) {
+#pragma unroll
+                for (int o = 1; o < (VEC ? IPT : 1); o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+            } else {
+                for (int o = 1; o < IP; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+            }
+            if (HEAD) dot *= decay;
+            const float u = live ? bs[t] * (vs[t * JB + jl] - dot) : 0.f;
+            float sum0 = 0.f, sum1 = 0.f;
+#pragma unroll
+            for (int r = 0; r < DS; ++r) {
+                S[r] = fmaf(kc[r], u, aS[r]);
+                if (r & 1) sum1 = fmaf(qc[r], S[r], sum1);
+                else sum0 = fmaf(qc[r], S[r], sum0);
+            }
+            return sum0 + sum1;
+        };
+        if (n == DC) {
+#pragma unroll
+            for (int t = 0; t < DC; ++t) part[t] = token(t);
+        } else {
+#pragma unroll
+            for (int t = 0; t < DC; ++t) part[t] = t < n ? token(t) : 0.f;
+        }
+        if (VEC) {
+            // tokens spread over the lanes while they are summed: a lane keeps one half of its tokens and hands the other on
+            int held = DC, first = 0;  // tokens this lane holds: first .. first + held - 1
+#pragma unroll
+            for (int o = IPT >> 1; o >= 1; o >>= 1) {
+                if (held > 1) {
+                    held >>= 1;
+                    const bool upper = (ipart & o) != 0;
+#pragma unroll
+                    for (int i = 0; i < DC / 2; ++i)
+                        if (i < held) {
+                            const float send = upper ? part[i] : part[i + held];
+                            const float keep = upper ? part[i + held] : part[i];
+                            part[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                        }
+                    if (upper) first += held;
+                } else {
+                    part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
+                }
+            }
+            constexpr int HELD = IPT > DC ? 1 : DC / (VEC ? IPT : 1);
+            if (live && (IPT <= DC || ipart % (IPT / DC > 0 ? IPT / DC : 1) == 0)) {
+#pragma unroll
+                for (int i = 0; i < HELD; ++i)
+                    if (first + i < n) g.out[(size_t)(t0 + first + i) * g.ldo + (size_t)h * Dv + j] = part[i];
+            }
+        } else {
 #pragma unroll
             for (int t = 0; t < DC; ++t)
-                if (t < n) out[(size_t)(t0 + t) * ldo + (size_t)h * Dv + j] = part[t];
+                for (int o = 1; o < IP; o <<= 1) part[t] += __shfl_xor_sync(0xffffffffu, part[t], o);
+            if (live && ipart == 0) {
+#pragma unroll
+                for (int t = 0; t < DC; ++t)
+                    if (t < n) g.out[(size_t)(t0 + t) * g.ldo + (size_t)h * Dv + j] = part[t];
+            }
         }
     }
     if (live) {
 #pragma unroll
-        for (int r = 0; r < DS; ++r) {
-            const int i = ipart + r * IP;
-            if (i < Dk) S_mem[i] = S[r];
-        }
+        for (int r = 0; r < DS; ++r)
+            if (owns(r)) S_mem[channel(r)] = S[r];
     }
 }
 
-// q, k [N, groups*Dk] (head h reads group h / heads_per_group), v [N, H*Dv], a [N, H*Dk] decays, beta [N, H]: float32,
-// unit column stride, any row stride.  out [N, H*Dv].
+// q, k [N, groups*Dk] (head h reads group h / heads_per_group), v [N, H*Dv], beta [N, H], decays a [N, H*Dk] or, with
+// head_decay, [N, H]: float32, unit column stride, any row stride.  out [N, H*Dv].
 extern "C" int cw_delta_scan(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* a, int lda,
-                             const float* beta, int ldb, float* state, long long state_stride, long long state_off,
+                             int head_decay, const float* beta, int ldb, float* state, long long state_stride, long long state_off,
                              const long long* slots, const int* tok_seq, const int* q_start, int S, int H, int Dk, int Dv,
-                             int heads_per_group, float* out, int ldo, cudaStream_t stream) {
+                             int heads_per_group, float* out, int ldo, const float* carry, int ldc, int C, int R, long long carry_off,
+                             cudaStream_t stream) {
     if (S == 0) return CW_OK;
     if (S < 0 || H <= 0 || Dk <= 0 || Dv <= 0 || heads_per_group <= 0 || H % heads_per_group) return CW_ERR_BAD_SIZE;
+    if (carry != nullptr && (C <= 0 || R < 0 || ldc < C)) return CW_ERR_BAD_SIZE;
     if (Dk > 32 * DS || H > 65535) return CW_ERR_UNSUPPORTED;
-    int IP = 1;
-    while (IP * DS < Dk) IP *= 2;
+    int IP = 1, log_ip = 0;
+    while (IP * DS < Dk) {
+        IP *= 2;
+        ++log_ip;
+    }
     int threads = 256;  // more value columns per block share the staged q, k and decays; fewer when a head has few columns
     while (threads > 32 && threads / IP >= 2 * Dv) threads /= 2;
     const int JB = threads / IP;
     dim3 grid(S, H, (Dv + JB - 1) / JB);
-    const int wide = Dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && lda % 4 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k & 15) == 0 &&
-                     ((uintptr_t)a & 15) == 0;
-    const size_t smem = 2 * sizeof(float) * (size_t)(3 * DC * Dk + DC * JB + DC);
-    static size_t allowed = 48 << 10;
-    if (smem > allowed) {
-        const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const int wide = Dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k & 15) == 0 &&
+                     (head_decay || (lda % 4 == 0 && ((uintptr_t)a & 15) == 0));
+    const bool vec = wide && Dk % DS == 0;
+    const size_t smem = 2 * sizeof(float) * (size_t)((head_decay ? 2 : 3) * DC * Dk + DC * JB + (head_decay ? 2 : 1) * DC);
+    using Kernel = void (*)(const DeltaScanArgs);
+    static const Kernel kernels[2][7] = {
+        {delta_scan_kernel<1, false>, delta_scan_kernel<2, false>, delta_scan_kernel<4, false>, delta_scan_kernel<8, false>,
+         delta_scan_kernel<16, false>, delta_scan_kernel<32, false>, delta_scan_kernel<0, false>},
+        {delta_scan_kernel<1, true>, delta_scan_kernel<2, true>, delta_scan_kernel<4, true>, delta_scan_kernel<8, true>,
+         delta_scan_kernel<16, true>, delta_scan_kernel<32, true>, delta_scan_kernel<0, true>}};
+    static size_t allowed[2][7] = {};
+    const int by_head = head_decay ? 1 : 0, which = vec ? log_ip : 6;
+    if (smem > (48u << 10) && smem > allowed[by_head][which]) {
+        const cudaError_t e = cudaFuncSetAttribute(kernels[by_head][which], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
-        allowed = smem;
+        allowed[by_head][which] = smem;
     }
-    return cw_launch_ordered(delta_scan_kernel, grid, dim3(threads), smem, stream, q, ldq, k, ldk, v, ldv, a, lda, beta, ldb, state,
-                             state_stride, state_off, slots, tok_seq, q_start, Dk, Dv, heads_per_group, IP, wide, out, ldo);
+    const DeltaScanArgs args = {q, ldq, k, ldk, v, ldv, a, lda, beta, ldb, state, state_stride, state_off, slots, tok_seq, q_start, Dk, Dv,
+                                heads_per_group, IP, wide, out, ldo, R > 0 ? carry : nullptr, ldc, C, R, carry_off};
+    return cw_launch_ordered(kernels[by_head][which], grid, dim3(threads), smem, stream, args);
 }
 
 // ---- the gates of a matrix memory -----------------------------------------------------------------------

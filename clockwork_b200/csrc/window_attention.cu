@@ -13,12 +13,14 @@
 //                        (`blocked`: positions are cut into blocks of `window` instead, and p sees the positions
 //                        of its own block up to itself; `sink`: a logit per head that enters the softmax's
 //                        denominator once, with no key and no value)
-//   cw_rotate_store      turns the leading entries of every query and key head by the token's position (entry i with
-//                        entry i + dims/2), writes the queries out and the rows [key | value] into the cache
+//   cw_rotate_store      turns the leading entries of every query and key head by the token's position (rotation.cuh),
+//                        writes the queries out and the rows [key | value] into the cache; before that, if asked, all of
+//                        the token's queries together are RMS-normed with a weight per entry, and all of its keys
 //   cw_pool_rows         for every token that ends a block of `pool` positions: the mean of the block's rows [key | value]
 //                        as the cache holds them, into the row of a second cache that the token's slot there names
 //   (window_merge_kernel adds up the parts of a token's window; only launched when windows are cut)
-// Further switches of cw_window_attention (WindowExtras; each usable alone): a window that never closes (window >= 2^30:
+// Further switches of cw_window_attention (each usable alone): `keep`: the first `keep` positions of the sequence stay
+// visible when the window has left them (a row's order of keys is then: kept positions before its window, its window); a window that never closes (window >= 2^30:
 // plain causal attention); `pool`: beside the window, every block of `pool` positions that ends at or before p - window is
 // seen as one key and value, read from the second cache (its rows come first in a row's order of keys); `softcap`: the
 // score (after the numbers per head) becomes cap tanh(score / cap); `slopes`: slope[h] (p - j) is taken off the (capped)
@@ -30,7 +32,7 @@
 // Scores, weights, the softmax statistics and the weighted sums are float32 in both run precisions; T names
 // the type of the product's output and of the cache.  A token's result depends on its position alone: keys
 // are taken in tiles that start at the window's first position, in order, whatever else the step holds.
-#include "common.cuh"
+#include "rotation.cuh"
 
 #define WA_MAX_COLS 16  // output columns per thread
 
@@ -66,34 +68,66 @@ extern "C" int cw_store_rows(const void* src, int ld, int col0, int width, void*
     return CW_ERR_BAD_DTYPE;
 }
 
-// src [N, ld] float32: a token's product row [queries (H*dk) | per key/value head: key (dk), value (dv)].  The first
-// `rot` entries of every query and key head are rotated: the pair (entry i, entry i + rot/2) by the angle
-// position * inv_freq[i], in float32.  Queries go to q_out [N, H*dk], the rows [key | value] to the cache row that the
-// token's slot names (slots null or < 0: nothing is stored).
-template <typename T>
+// src [N, ld] float32: a token's product row [queries (H*dk) | per key/value head: key (dk), value (dv)].  With q_norm
+// [H*dk] and k_norm [G*dk] the queries are first divided by the root mean square (eps inside the root) of all H*dk of them
+// and multiplied by q_norm, the keys likewise over their G*dk entries.  Then the leading entries of every query and key
+// head are rotated, everything in float32.  Queries go to q_out [N, H*dk], the rows [key | value] to the cache row that
+// the token's slot names (slots null or < 0: nothing is stored).
+template <typename T, bool NORM>
 __global__ void __launch_bounds__(256)
 rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict__ positions, const int* __restrict__ tok_seq,
-                    const int* __restrict__ slots, const float* __restrict__ inv_freq, int H, int G, int dk, int dv, int rot,
-                    T* __restrict__ q_out, T* __restrict__ cache, long long total_rows, int* __restrict__ status) {
+                    const int* __restrict__ slots, Rotation rot, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
+                    float eps, int H, int G, int dk, int dv, T* __restrict__ q_out, T* __restrict__ cache, long long total_rows,
+                    int* __restrict__ status) {
+    extern __shared__ float rs_table[];  // cosines, then sines, of the token's pairs
+    __shared__ float scratch[33];
     pdl_wait();
     const int n = blockIdx.x;
-    const int HQ = H * dk, row = dk + dv, half = rot >> 1;
+    const int HQ = H * dk, row = dk + dv, half = rot.dims >> 1;
     T* qo = q_out + (size_t)n * HQ;
     if (tok_seq[n] < 0) {  // padding of a fixed-shape step
         for (int c = threadIdx.x; c < HQ; c += blockDim.x) qo[c] = from_f<T>(0.f);
         return;
     }
-    const float p = (float)positions[n];
     const float* x = src + (size_t)n * ld;
-    auto turned = [&](const float* head, int i) {  // entry i (< rot) of a head after the rotation
-        const int j = i < half ? i : i - half;
-        float sn, cs;
-        sincosf(p * inv_freq[j], &sn, &cs);
-        return i < half ? head[i] * cs - head[i + half] * sn : head[i] * cs + head[i - half] * sn;
+    const float* kv = x + HQ;
+    float* cs = rs_table;
+    float* sn = rs_table + half;
+    rotation_table(rot, positions[n], cs, sn);
+    float q_inv = 1.f, k_inv = 1.f;
+    if (NORM) {
+        float qs = 0.f, ks = 0.f;
+        for (int c = threadIdx.x; c < HQ; c += blockDim.x) qs = fmaf(x[c], x[c], qs);
+        for (int g = 0; g < G; ++g)
+            for (int i = threadIdx.x; i < dk; i += blockDim.x) {
+                const float k = kv[(size_t)g * row + i];
+                ks = fmaf(k, k, ks);
+            }
+        q_inv = 1.0f / sqrtf(block_sum(qs, scratch) / (float)HQ + eps);
+        k_inv = 1.0f / sqrtf(block_sum(ks, scratch) / (float)(G * dk) + eps);
+    }
+    __syncthreads();  // the table is written
+    // entry i of a head after norm and rotation (w: the norm's weights of this head)
+    auto entry = [&](const float* head, const float* w, float inv, int i) {
+        auto normed = [&](int e) { return NORM ? head[e] * inv * w[e] : head[e]; };
+        if (i >= rot.dims) return normed(i);
+        int pair, other;
+        bool first;
+        if (rot.interleaved) {
+            pair = i >> 1;
+            other = i ^ 1;
+            first = (i & 1) == 0;
+        } else {
+            first = i < half;
+            pair = first ? i : i - half;
+            other = first ? i + half : i - half;
+        }
+        const float a = normed(i), b = normed(other);
+        return first ? a * cs[pair] - b * sn[pair] : a * cs[pair] + b * sn[pair];
     };
     for (int c = threadIdx.x; c < HQ; c += blockDim.x) {
         const int h = c / dk, i = c - h * dk;
-        qo[c] = from_f<T>(i < rot ? turned(x + (size_t)h * dk, i) : x[c]);
+        qo[c] = from_f<T>(entry(x + (size_t)h * dk, NORM ? q_norm + (size_t)h * dk : nullptr, q_inv, i));
     }
     const int slot = slots != nullptr ? slots[n] : -1;
     if (slot < 0) return;
@@ -102,28 +136,36 @@ rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict
         return;
     }
     T* to = cache + (size_t)slot * G * row;
-    const float* kv = x + HQ;
     for (int c = threadIdx.x; c < G * row; c += blockDim.x) {
         const int g = c / row, i = c - g * row;
-        to[c] = from_f<T>(i < rot ? turned(kv + (size_t)g * row, i) : kv[c]);
+        to[c] = from_f<T>(i < dk ? entry(kv + (size_t)g * row, NORM ? k_norm + (size_t)g * dk : nullptr, k_inv, i) : kv[c]);
     }
 }
 
 extern "C" int cw_rotate_store(const float* src, int ld, const int* positions, const int* tok_seq, const int* slots,
-                               const float* inv_freq, int N, int H, int G, int dk, int dv, int rot, void* q_out, void* cache,
+                               const float* inv_freq, int rot_dims, int interleaved, float amplitude, const float* q_norm,
+                               const float* k_norm, float eps, int N, int H, int G, int dk, int dv, void* q_out, void* cache,
                                long long total_rows, int dtype, int* status, cudaStream_t stream) {
     if (N == 0) return CW_OK;
-    if (N < 0 || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || rot < 0 || rot > dk || (rot & 1) || ld < H * dk + G * (dk + dv) ||
-        (rot > 0 && inv_freq == nullptr) || total_rows < 0)
+    const Rotation rot = {inv_freq, rot_dims, interleaved, amplitude};
+    if (N < 0 || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || !rotation_ok(rot, dk) || ld < H * dk + G * (dk + dv) || total_rows < 0 ||
+        (q_norm == nullptr) != (k_norm == nullptr))
         return CW_ERR_BAD_SIZE;
+    if (rot_dims > 8192) return CW_ERR_UNSUPPORTED;
     int threads = 64;
     while (threads < 256 && threads < H * dk) threads *= 2;
-    if (dtype == 0)
-        return cw_launch_ordered(rotate_store_kernel<float>, dim3(N), dim3(threads), 0, stream, src, ld, positions, tok_seq, slots, inv_freq,
-                                 H, G, dk, dv, rot, (float*)q_out, (float*)cache, total_rows, status);
-    if (dtype == 1)
-        return cw_launch_ordered(rotate_store_kernel<bf16>, dim3(N), dim3(threads), 0, stream, src, ld, positions, tok_seq, slots, inv_freq,
-                                 H, G, dk, dv, rot, (bf16*)q_out, (bf16*)cache, total_rows, status);
+    const size_t smem = sizeof(float) * (size_t)rot_dims;
+    const dim3 grid(N), block(threads);
+    if (dtype == 0) {
+        const auto kernel = q_norm != nullptr ? rotate_store_kernel<float, true> : rotate_store_kernel<float, false>;
+        return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv,
+                                 (float*)q_out, (float*)cache, total_rows, status);
+    }
+    if (dtype == 1) {
+        const auto kernel = q_norm != nullptr ? rotate_store_kernel<bf16, true> : rotate_store_kernel<bf16, false>;
+        return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv,
+                                 (bf16*)q_out, (bf16*)cache, total_rows, status);
+    }
     return CW_ERR_BAD_DTYPE;
 }
 
@@ -234,6 +276,7 @@ struct WindowAttentionArgs {
     const void* pool_cache;   // [rows, G, dk + dv]: row b of a request is the mean of its positions b*pool .. b*pool + pool - 1
     const int* pool_tables;   // [S, pool_max_blocks]
     int pool_max_blocks, pool_pages;
+    int keep;                 // the sequence's first `keep` positions are seen by every later one
 };
 
 // how many pooled blocks position p sees: those that end at or before p - window
@@ -241,6 +284,8 @@ __device__ __forceinline__ int wa_pooled_blocks(int p, int window, int pool) {
     const int behind = p - window + 1;  // positions before the window
     return pool > 0 && behind > 0 ? behind / pool : 0;
 }
+// how many kept positions lie before a window that starts at `first`
+__device__ __forceinline__ int wa_kept_before(int first, int keep) { return min(first, keep); }
 __device__ __forceinline__ float wa_query_temperature(int p, float coef, int every) {
     return every > 0 ? 1.f + coef * logf((float)((p + 1) / every + 1)) : 1.f;
 }
@@ -263,8 +308,9 @@ window_attention_kernel(const WindowAttentionArgs a) {
     }
     const int p = a.positions[n];
     const int first = a.blocked ? p - p % a.window : max(0, p - a.window + 1);
-    // the row's keys in one order: its pooled blocks 0 .. nb-1, then the positions first .. p
-    const int nb = wa_pooled_blocks(p, a.window, a.pool);
+    // the row's keys in one order: its pooled blocks 0 .. nb-1 (or the kept positions 0 .. nb-1 before its window), then
+    // the positions first .. p
+    const int nb = a.keep > 0 ? wa_kept_before(first, a.keep) : wa_pooled_blocks(p, a.window, a.pool);
     const int lo = part * a.part_keys;
     const int total = nb + p + 1 - first;
     const int hi = part == a.parts - 1 ? total : min(total, lo + a.part_keys);  // keys lo .. hi-1 of that order (the last part: all the rest)
@@ -301,7 +347,7 @@ window_attention_kernel(const WindowAttentionArgs a) {
             int row = -1, back = 0;
             if (tid < nk) {
                 const int v = j0 + tid;
-                if (v < nb) {  // a pooled block
+                if (v < nb && a.keep == 0) {  // a pooled block
                     const int blk = v / a.page_size;
                     const int page = blk < a.pool_max_blocks ? pool_table[blk] : -1;
                     if (page < 0 || page >= a.pool_pages)
@@ -310,7 +356,7 @@ window_attention_kernel(const WindowAttentionArgs a) {
                         row = page * a.page_size + v % a.page_size;
                     back = -1;
                 } else {
-                    const int pos = first + (v - nb), blk = pos / a.page_size;
+                    const int pos = v < nb ? v : first + (v - nb), blk = pos / a.page_size;
                     const int page = blk < a.max_blocks ? table[blk] : -1;
                     if (page < 0 || page >= a.num_pages)
                         cw_report(a.status, CW_ST_PAGE_RANGE, n, page);
@@ -422,7 +468,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 window_merge_kernel(const float* __restrict__ partial, const int* __restrict__ positions, const int* __restrict__ tok_seq,
                     int H, int dv, int window, int parts, int part_keys, int sigmoid_weights, int all_parts, int blocked,
-                    const float* __restrict__ sink, T* __restrict__ out, int pool, const float* __restrict__ gate, int ldg) {
+                    const float* __restrict__ sink, T* __restrict__ out, int pool, int keep, const float* __restrict__ gate, int ldg) {
     __shared__ float factor[64];
     __shared__ float denominator;
     pdl_wait();
@@ -430,7 +476,8 @@ window_merge_kernel(const float* __restrict__ partial, const int* __restrict__ p
     if (tok_seq[n] < 0) return;  // (the attention kernel wrote the zeros)
     const int HV = H * dv, stride = HV + 2 * H;
     const int p = positions[n];
-    const int keys = (blocked ? p % window + 1 : p + 1 - max(0, p - window + 1)) + wa_pooled_blocks(p, window, pool);
+    const int keys = (blocked ? p % window + 1 : p + 1 - max(0, p - window + 1)) +
+                     (keep > 0 ? wa_kept_before(max(0, p - window + 1), keep) : wa_pooled_blocks(p, window, pool));
     const int used = all_parts ? parts : min(parts, (keys + part_keys - 1) / part_keys);  // (parts that hold none of the row's keys add nothing)
     const float* base = partial + (size_t)n * parts * stride;
     if (threadIdx.x == 0) {
@@ -550,10 +597,15 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
     const int h = g0 * per + warp;  // this warp's query head
     const int gl = warp / per;      // its key/value head among the block's
     const int p0 = a.positions[row0];
-    const int first = a.blocked ? p0 - p0 % a.window : max(0, p0 - a.window + 1);
-    // What the tile's rows see, in key tiles of 32: the pooled blocks 0 .. NB-1 that its last row sees (tiles 0 .. pool_tiles-1,
-    // the last of them part empty), then the positions first .. p0 + rows - 1; `parts` equal runs of whole key tiles.
-    const int NB = wa_pooled_blocks(p0 + rows - 1, a.window, a.pool);
+    int first = a.blocked ? p0 - p0 % a.window : max(0, p0 - a.window + 1);
+    // (a window that starts within the kept positions simply starts at 0; with a gap between the two, the pages of the gap
+    // may have been given back)
+    if (a.keep > 0 && first <= a.keep) first = 0;
+    // What the tile's rows see, in key tiles of 32: the pooled blocks 0 .. NB-1 that its last row sees, or the kept positions
+    // 0 .. NB-1 before `first` (tiles 0 .. pool_tiles-1, the last of them part empty), then the positions first .. p0 + rows - 1;
+    // `parts` equal runs of whole key tiles.
+    const bool kept = a.keep > 0;
+    const int NB = kept ? wa_kept_before(first, a.keep) : wa_pooled_blocks(p0 + rows - 1, a.window, a.pool);
     const int pool_tiles = (NB + WM_BN - 1) / WM_BN;
     const int all_tiles = pool_tiles + (p0 + rows - first + WM_BN - 1) / WM_BN;
     const int part_tiles = (all_tiles + a.parts - 1) / a.parts;
@@ -623,8 +675,12 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
         const bf16* from = cache;
         if (t < pool_tiles) {
             const int b = t * WM_BN + j;
-            if (b < NB) page = pool_page_of(b, offset);
-            from = pool_cache;
+            if (kept) {
+                if (b < NB) page = page_of(b, offset);
+            } else {
+                if (b < NB) page = pool_page_of(b, offset);
+                from = pool_cache;
+            }
         } else {
             const int pos = first + (t - pool_tiles) * WM_BN + j;
             if (pos < hi) page = page_of(pos, offset);
@@ -659,12 +715,12 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
     for (int x = 0; x < 2; ++x) {
         const int p = p0 + r_lo + 8 * x;
         row_first[x] = a.blocked ? p - p % a.window : p - a.window + 1;
-        row_blocks[x] = wa_pooled_blocks(p, a.window, a.pool);
+        row_blocks[x] = kept ? NB : wa_pooled_blocks(p, a.window, a.pool);
         row_temp[x] = wa_query_temperature(p, a.temp_coef, a.temp_every);
     }
     const bool bent = a.softcap > 0.f || a.slopes != nullptr || a.temp_every > 0;  // scores that are more than scaled and shifted
     const float slope = a.slopes != nullptr ? a.slopes[h] : 0.f;
-    const int first_blocks = wa_pooled_blocks(p0, a.window, a.pool);  // pooled blocks that every row of the tile sees
+    const int first_blocks = kept ? NB : wa_pooled_blocks(p0, a.window, a.pool);  // pooled blocks (kept positions) that every row of the tile sees
     const int last_first = a.blocked ? (p0 + 15) - (p0 + 15) % a.window : p0 + 15 - a.window + 1;  // of the tile's last row
     const float head_scale = a.head_scale != nullptr ? a.head_scale[h] : 1.f;
     const float head_bias = a.head_bias != nullptr ? a.head_bias[h] : 0.f;
@@ -741,14 +797,15 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
                 if (!whole) {
                     const int row = r_lo + (e >> 1) * 8;
                     const int p = p0 + row;
-                    on = pooled ? row < rows && j < row_blocks[e >> 1] : row < rows && j <= p && j >= row_first[e >> 1] && j < hi;
+                    on = pooled ? row < rows && j < row_blocks[e >> 1]
+                                : row < rows && j <= p && (j >= row_first[e >> 1] || j < a.keep) && j < hi;
                 }
                 float v = s[nt][e];
                 if (bent) v *= row_temp[e >> 1];
                 v = fmaf(v, head_scale, head_bias);
                 if (bent) {
                     if (a.softcap > 0.f) v = a.softcap * tanhf(v / a.softcap);
-                    if (!pooled) v -= slope * (float)(p0 + r_lo + (e >> 1) * 8 - j);
+                    if (!pooled || kept) v -= slope * (float)(p0 + r_lo + (e >> 1) * 8 - j);
                 }
                 v = on ? v : -INFINITY;
                 s[nt][e] = v;
@@ -905,11 +962,12 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
                                    void* out, int parts, float* partial, const int* q_start, int S, int dtype, int* status,
                                    float softcap, const float* slopes, float temp_coef, int temp_every, const float* gate, int ldg,
                                    int pool, const void* pool_cache, const int* pool_tables, int pool_max_blocks, int pool_pages,
-                                   cudaStream_t stream) {
+                                   int keep, cudaStream_t stream) {
     if (N == 0) return CW_OK;
     if (softcap < 0.f || temp_every < 0 || pool < 0 || (gate != nullptr && ldg < H)) return CW_ERR_BAD_SIZE;
     if (pool > 0 && (pool_cache == nullptr || pool_tables == nullptr || pool_max_blocks <= 0 || pool_pages <= 0 || blocked || slopes != nullptr))
         return CW_ERR_BAD_SIZE;  // (a pooled block has no distance, and blocks of positions have nothing before them)
+    if (keep < 0 || (keep > 0 && (blocked || pool > 0))) return CW_ERR_BAD_SIZE;  // (kept positions lie before a plain window)
     if (N < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || window <= 0 || page_size <= 0 || max_blocks <= 0 ||
         ldq < H * dk || parts < 1)
         return CW_ERR_BAD_SIZE;
@@ -922,14 +980,14 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
         const WindowAttentionArgs base = {q, ldq, cache, block_tables, max_blocks, page_size, num_pages, positions, tok_seq, H, G, dk, dv,
                                           window, scale, head_scale, talk, head_bias, sigmoid_weights, blocked, sink, out, WM_BN, parts, 0,
                                           partial, status, softcap, slopes, temp_coef, temp_every, gate, ldg, pool, pool_cache, pool_tables,
-                                          pool_max_blocks, pool_pages};
+                                          pool_max_blocks, pool_pages, keep};
         int launched = 0;
         const int rc = window_attention_mma(base, q_start, S, N, stream, &launched);
         if (rc != 0) return rc;
         if (launched) {
             if (parts == 1) return CW_OK;
             return cw_launch_ordered(window_merge_kernel<bf16>, dim3(N, H), dim3(merge_threads), 0, stream, (const float*)partial, positions, tok_seq, H,
-                                     dv, window, parts, 0, sigmoid_weights, 1, blocked, sink, (bf16*)out, pool, gate, ldg);
+                                     dv, window, parts, 0, sigmoid_weights, 1, blocked, sink, (bf16*)out, pool, keep, gate, ldg);
         }
     }
     int threads = 128;
@@ -945,13 +1003,13 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
     if (smem > (200u << 10)) return CW_ERR_UNSUPPORTED;
     // (a row's order of keys is cut in `parts` runs: float32 runs never cut, so the longest row that a cut must cover is a
     // window and the pooled blocks before it; a window that never closes is cut as if it held 2^20 keys)
-    const long long longest = (long long)min(window, 1 << 20) + (pool > 0 ? (1 << 20) / pool : 0);
+    const long long longest = (long long)min(window, 1 << 20) + (pool > 0 ? (1 << 20) / pool : 0) + keep;
     int part_keys = (int)((longest + parts - 1) / parts);
     part_keys = (part_keys + tile - 1) / tile * tile;
     WindowAttentionArgs a = {q, ldq, cache, block_tables, max_blocks, page_size, num_pages, positions, tok_seq, H, G, dk, dv,
                              window, scale, head_scale, talk, head_bias, sigmoid_weights, blocked, sink, out, tile, parts, part_keys,
                              partial, status, softcap, slopes, temp_coef, temp_every, gate, ldg, pool, pool_cache, pool_tables,
-                             pool_max_blocks, pool_pages};
+                             pool_max_blocks, pool_pages, keep};
     static size_t allowed[2] = {48 << 10, 48 << 10};
     if (dtype != 0 && dtype != 1) return CW_ERR_BAD_DTYPE;
     if (smem > allowed[dtype]) {
@@ -967,9 +1025,9 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
     if (rc != 0 || parts == 1) return rc;
     if (dtype == 0)
         return cw_launch_ordered(window_merge_kernel<float>, dim3(N, H), dim3(merge_threads), 0, stream, (const float*)partial, positions, tok_seq,
-                                 H, dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (float*)out, pool, gate, ldg);
+                                 H, dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (float*)out, pool, keep, gate, ldg);
     return cw_launch_ordered(window_merge_kernel<bf16>, dim3(N, H), dim3(merge_threads), 0, stream, (const float*)partial, positions, tok_seq, H,
-                             dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (bf16*)out, pool, gate, ldg);
+                             dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (bf16*)out, pool, keep, gate, ldg);
 }
 
 CW_TRACE_TU(window_attention)

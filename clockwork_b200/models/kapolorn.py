@@ -63,6 +63,20 @@ def _layers_2k(repeats: int) -> list:
     return [pair, pair, pair, delta] * repeats
 
 
+def _loop_bounds(loop, layers: int) -> tuple:
+    """(start, stop, times) of config.json's ``loop`` over a list of ``layers`` layers; None: no loop."""
+    if loop is None:
+        return (0, 0, 1)
+    start, stop = loop.get("start"), loop.get("stop")
+    for key, value in (("start", start), ("stop", stop)):
+        if isinstance(value, bool) or not isinstance(value, int) or value < 0:
+            raise ValueError(f"config.json: loop.{key} must be a non-negative integer, got {value!r}")
+    times = _need(loop, "times", "loop")
+    if not start <= stop <= layers:
+        raise ValueError(f"config.json: a loop over layers {start} .. {stop - 1} does not fit {layers} layers")
+    return (start, stop, times)
+
+
 class KapolornArchitecture:
     name = "Kapolorn"
     layer_count_key = None  # the layers are a list: a shape with fewer layers is another list
@@ -137,18 +151,8 @@ class KapolornArchitecture:
             where = f"layers[{i}]"
             layers.append((self._mixer(entry.get("type"), entry.get("mixer") or {}, width, eps, where + ".mixer"),
                            self._ffn(entry.get("mlp"), width, where + ".mlp")))
-        loop = raw.get("loop")
-        if loop is None:
-            bounds = (0, 0, 1)
-        else:
-            start, stop = loop.get("start"), loop.get("stop")
-            for key, value in (("start", start), ("stop", stop)):
-                if isinstance(value, bool) or not isinstance(value, int) or value < 0:
-                    raise ValueError(f"config.json: loop.{key} must be a non-negative integer, got {value!r}")
-            bounds = (start, stop, _need(loop, "times", "loop"))
-            if not start <= stop <= len(layers):
-                raise ValueError(f"config.json: a loop over layers {start} .. {stop - 1} does not fit {len(layers)} layers")
-        return KapolornConfig(_need(raw, "vocab", "the model"), width, eps, scale, cap, bounds, tuple(layers), dict(raw))
+        return KapolornConfig(_need(raw, "vocab", "the model"), width, eps, scale, cap, _loop_bounds(raw.get("loop"), len(layers)),
+                              tuple(layers), dict(raw))
 
     def model_spec(self, config: KapolornConfig) -> ModelSpec:
         norm = PartSpec("rmsnorm", {"size": config.width, "eps": config.eps, "weight_suffix": ""})

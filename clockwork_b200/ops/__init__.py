@@ -242,10 +242,10 @@ def depth_average(x: torch.Tensor, terms, history: torch.Tensor, index: int, coe
     return normed
 
 
-def softcap_(x: torch.Tensor, cap: float) -> torch.Tensor:
-    """In place on float32 ``x``: ``cap * tanh(x / cap)``."""
+def softcap_(x: torch.Tensor, cap: float | None, scale: float = 1.0) -> torch.Tensor:
+    """In place on float32 ``x``: ``cap * tanh(scale * x / cap)`` (``cap`` None: ``scale * x``)."""
     _need(x, torch.float32, "x")
-    check(library().cw_softcap(_ptr(x), x.numel(), float(cap), _stream()), "softcap")
+    check(library().cw_softcap(_ptr(x), x.numel(), float(cap or 0.0), float(scale), _stream()), "softcap")
     return x
 
 
@@ -261,20 +261,22 @@ class PartialSums:
 
 
 def _add_partial_sums(resid: torch.Tensor, parts: PartialSums, weight: torch.Tensor | None, eps: float,
-                      out: torch.Tensor | None) -> None:
+                      out: torch.Tensor | None, center: bool = False) -> None:
     _need(parts.slabs, torch.float32, "partial sums", 3)
     n, h = resid.shape
     splits, slab_rows, width = parts.slabs.shape
     if width != h or parts.rows != n or slab_rows < n:
         raise ValueError(f"partial sums {tuple(parts.slabs.shape)} of {parts.rows} rows do not match residual {tuple(resid.shape)}")
     check(library().cw_add_parts_rmsnorm(_ptr(resid), _ptr(parts.slabs), splits, slab_rows, _ptr(weight), _ptr(out), n, h,
-                                         float(eps), 0 if out is None else dtype_code(out.dtype), _stream()), "add_parts_rmsnorm")
+                                         float(eps), 1 if center else 0, 0 if out is None else dtype_code(out.dtype), _stream()),
+          "add_parts_rmsnorm")
 
 
 def add_rmsnorm(resid: torch.Tensor, delta, weight: torch.Tensor, eps: float,
-                out_dtype: torch.dtype, status: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+                out_dtype: torch.dtype, status: torch.Tensor, out: torch.Tensor | None = None, center: bool = False) -> torch.Tensor:
     """``resid += delta`` (if given: a tensor, or the ``PartialSums`` of a product), then returns
-    ``weight * rmsnorm(resid)`` as ``out_dtype``."""
+    ``weight * rmsnorm(resid)`` as ``out_dtype``.  ``center``: layer norm, the row's mean taken off first
+    (``(x - mean) / sqrt(mean of the squared deviations + eps) * weight``)."""
     _need(resid, torch.float32, "resid", 2)
     _need(weight, torch.float32, "weight", 1)
     n, h = resid.shape
@@ -283,7 +285,7 @@ def add_rmsnorm(resid: torch.Tensor, delta, weight: torch.Tensor, eps: float,
     if isinstance(delta, PartialSums):
         if out is None:
             out = torch.empty((n, h), dtype=out_dtype, device=resid.device)
-        _add_partial_sums(resid, delta, weight, eps, out)
+        _add_partial_sums(resid, delta, weight, eps, out, center)
         return out
     if delta is not None:
         _need(delta, out_dtype, "delta", 2)
@@ -292,13 +294,13 @@ def add_rmsnorm(resid: torch.Tensor, delta, weight: torch.Tensor, eps: float,
     if out is None:
         out = torch.empty((n, h), dtype=out_dtype, device=resid.device)
     check(library().cw_add_rmsnorm(_ptr(resid), _ptr(delta), _ptr(weight), _ptr(out), None, n, n, h, float(eps),
-                                   dtype_code(out_dtype), _ptr(status), _stream()), "add_rmsnorm")
+                                   1 if center else 0, dtype_code(out_dtype), _ptr(status), _stream()), "add_rmsnorm")
     return out
 
 
 def rmsnorm_rows(resid: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, eps: float,
-                 out_dtype: torch.dtype, status: torch.Tensor) -> torch.Tensor:
-    """``weight * rmsnorm(resid[rows])`` as ``out_dtype`` [R, H]."""
+                 out_dtype: torch.dtype, status: torch.Tensor, center: bool = False) -> torch.Tensor:
+    """``weight * rmsnorm(resid[rows])`` as ``out_dtype`` [R, H] (``center``: layer norm)."""
     _need(resid, torch.float32, "resid", 2)
     _need(rows, torch.int32, "rows", 1)
     _need(weight, torch.float32, "weight", 1)
@@ -306,7 +308,7 @@ def rmsnorm_rows(resid: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, 
     r = rows.shape[0]
     out = torch.empty((r, h), dtype=out_dtype, device=resid.device)
     check(library().cw_add_rmsnorm(_ptr(resid), None, _ptr(weight), _ptr(out), _ptr(rows), r, n, h, float(eps),
-                                   dtype_code(out_dtype), _ptr(status), _stream()), "rmsnorm_rows")
+                                   1 if center else 0, dtype_code(out_dtype), _ptr(status), _stream()), "rmsnorm_rows")
     return out
 
 

@@ -133,10 +133,67 @@ def delta_scan(q, k, v, pre, beta, dt_bias, a_log, view, offset: int, ctx, heads
 
     check(library().cw_delta_coefficients(_ptr(pre), ld(pre), _ptr(dt_bias), _ptr(a_log), _ptr(beta), ld(beta), n, heads, dk, _stream()),
           "delta_coefficients")
-    check(library().cw_delta_scan(_ptr(q), ld(q), _ptr(k), ld(k), _ptr(v), ld(v), _ptr(pre), ld(pre), _ptr(beta), ld(beta), state, stride,
+    check(library().cw_delta_scan(_ptr(q), ld(q), _ptr(k), ld(k), _ptr(v), ld(v), _ptr(pre), ld(pre), 0, _ptr(beta), ld(beta), state, stride,
                                   offset, slots, _ptr(ctx.tok_seq), _ptr(ctx.q_start), ctx.num_seqs, heads, dk, dv, heads_per_group,
-                                  _ptr(out), heads * dv, _stream()), "delta_scan")
+                                  _ptr(out), heads * dv, None, 0, 0, 0, 0, _stream()), "delta_scan")
     return out
+
+
+def head_delta(x, conv_weight, beta, decay, dt_bias, a_log, view, scan_offset: int, conv_offset: int, ctx, groups: int, heads: int,
+               dk: int, dv: int, unit_eps: float, q_scale: float) -> torch.Tensor:
+    """float32 [N, heads*dv]: everything between a delta layer's joint product and its output norm, for one decay per head.
+    ``x`` [N, >= 2*groups*dk + heads*dv] holds ``[q | k | v | ..]``; these columns pass a causal convolution of ``taps`` taps per
+    channel (``conv_weight`` [channels, taps], the current token's last) and SiLU; q and k heads are divided by
+    ``sqrt(sum of squares + unit_eps)``, q also multiplied by ``q_scale``; ``beta = sigmoid(beta)`` and
+    ``g = exp(-exp(a_log) softplus(decay + dt_bias))`` per head; per head ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; y = S^T q``.
+    The state piece at ``scan_offset`` holds S, the one at ``conv_offset`` the convolutions' last taps-1 inputs (both are
+    carried on).  Two kernels."""
+    for name, t in (("x", x), ("beta", beta), ("decay", decay)):
+        if t.dtype != torch.float32 or t.dim() != 2 or t.stride(1) != 1:
+            raise ValueError(f"{name} must be float32 [N, *] with unit column stride")
+    _need(conv_weight, torch.float32, "conv weight", 2)
+    _need(dt_bias, torch.float32, "dt_bias", 1)
+    _need(a_log, torch.float32, "a_log", 1)
+    n, qk = x.shape[0], groups * dk
+    channels = 2 * qk + heads * dv
+    if conv_weight.shape[0] != channels or x.shape[1] < channels or heads % groups:
+        raise ValueError(f"x {tuple(x.shape)} and conv weight {tuple(conv_weight.shape)} do not hold {channels} channels")
+    if dt_bias.shape[0] != heads or a_log.shape[0] != heads or beta.shape[1] != heads or decay.shape[1] != heads:
+        raise ValueError(f"beta, decay, dt_bias and a_log must have {heads} entries")
+    taps = conv_weight.shape[1]
+    out = torch.empty((n, heads * dv), dtype=torch.float32, device=x.device)
+    qkv = torch.empty((n, channels), dtype=torch.float32, device=x.device)
+    coef = torch.empty((n, 2 * heads), dtype=torch.float32, device=x.device)  # [decay | beta]
+    state, stride, slots = _state_args(view)
+
+    def ld(t):
+        return t.stride(0) if n > 1 else max(t.stride(0), t.shape[1])
+
+    check(library().cw_delta_prepare(_ptr(x), ld(x), _ptr(conv_weight), taps, state, stride, conv_offset, slots, _ptr(ctx.tok_seq),
+                                     _ptr(ctx.q_start), groups, dk, heads, dv, float(unit_eps), float(q_scale), _ptr(beta), ld(beta),
+                                     _ptr(decay), ld(decay), _ptr(dt_bias), _ptr(a_log), n, _ptr(qkv), _ptr(coef), _stream()), "delta_prepare")
+    check(library().cw_delta_scan(_ptr(qkv), channels, _ptr(qkv[:, qk:]), channels, _ptr(qkv[:, 2 * qk :]), channels, _ptr(coef), 2 * heads, 1,
+                                  _ptr(coef[:, heads:]), 2 * heads, state, stride, scan_offset, slots, _ptr(ctx.tok_seq), _ptr(ctx.q_start),
+                                  ctx.num_seqs, heads, dk, dv, heads // groups, _ptr(out), heads * dv, _ptr(x), ld(x), channels, taps - 1,
+                                  conv_offset, _stream()), "delta_scan")
+    return out
+
+
+def rotate_heads_(x: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, heads: int, dim: int, dims: int,
+                  interleaved: bool = False, amplitude: float = 1.0) -> torch.Tensor:
+    """In place on the first ``heads*dim`` columns of float32 ``x`` [N, C]: the first ``dims`` entries of every head turned by
+    the token's position, entry i with entry i + dims/2 (``interleaved``: entry 2i with entry 2i + 1) by the float32 angle
+    ``position * inv_freq[i]``, sines and cosines times ``amplitude``."""
+    if x.dtype != torch.float32 or x.dim() != 2 or x.stride(1) != 1 or x.shape[1] < heads * dim:
+        raise ValueError("x must be float32 [N, >= heads*dim] with unit column stride")
+    _need(positions, torch.int32, "positions", 1)
+    _need(inv_freq, torch.float32, "inv_freq", 1)
+    n = x.shape[0]
+    if inv_freq.shape[0] * 2 != dims or positions.shape[0] < n:
+        raise ValueError("inv_freq needs an entry per rotated pair, positions one per row")
+    check(library().cw_rotate_heads(_ptr(x), x.stride(0) if n > 1 else max(x.stride(0), x.shape[1]), _ptr(positions), _ptr(inv_freq), dims,
+                                    1 if interleaved else 0, float(amplitude), n, heads, dim, _stream()), "rotate_heads")
+    return x
 
 
 def gate_scan(zi: torch.Tensor, zf: torch.Tensor, bias_i: torch.Tensor | None, bias_f: torch.Tensor | None, cap: float, view,
@@ -214,19 +271,20 @@ def activation_cols_(x: torch.Tensor, cols: int, kind: int) -> torch.Tensor:
     return x
 
 
-def gated_group_norm(y: torch.Tensor, z: torch.Tensor | None, weight: torch.Tensor, parts: int, eps: float, gate_first: bool,
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor | None, weight: torch.Tensor | None, parts: int, eps: float, gate_first: bool,
                      out_dtype: torch.dtype, gate: int = GATE_SILU, shared_weight: bool = False) -> torch.Tensor:
     """``gate_first``: norm_parts(y * gate(z)) * weight; else norm_parts(y) * weight * gate(z).  y, z float32.
     ``gate``: silu or sigmoid, or ``GATE_NONE`` (``z`` None: norm_parts(y) * weight).  ``shared_weight``: ``weight`` has one
-    part's width and every part uses it."""
+    part's width and every part uses it.  ``weight`` None: there is none to multiply by."""
     _need(y, torch.float32, "y", 2)
     if (z is None) != (gate == GATE_NONE):
         raise ValueError("GATE_NONE goes with z = None")
     if z is not None and (z.dtype != torch.float32 or z.dim() != 2 or z.stride(1) != 1):
         raise ValueError("z must be float32 [N, C] with unit column stride")
-    _need(weight, torch.float32, "weight", 1)
     n, c = y.shape
-    if weight.shape[0] != (c // parts if shared_weight else c):
+    if weight is not None:
+        _need(weight, torch.float32, "weight", 1)
+    if weight is not None and weight.shape[0] != (c // parts if shared_weight else c):
         raise ValueError(f"weight of {weight.shape[0]} for {parts} parts of {c} columns")
     out = torch.empty((n, c), dtype=out_dtype, device=y.device)
     mode = (1 if gate_first else 0) | (2 if gate == GATE_SIGMOID else 0) | (4 if shared_weight else 0) | (8 if z is None else 0)

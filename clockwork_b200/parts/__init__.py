@@ -2,7 +2,7 @@
 Importing this package registers the built-in kinds."""
 
 from . import (  # noqa: F401  (registration)
-    attention, block, depth_block, feedforward, latent_attention, pair_embedding, parallel_block, rmsnorm, rotary, side_by_side,
+    attention, block, depth_block, feedforward, latent_attention, layernorm, pair_embedding, parallel_block, rmsnorm, rotary, side_by_side,
     state_mixers, swiglu, window_attention,
 )
 from .base import (

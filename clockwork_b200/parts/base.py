@@ -41,7 +41,8 @@ class PagedKVNeed:
     keys and values; 1 for a mixer that keeps one row per token (a latent that keys and values are both
     made from): its view's ``k_cache`` and ``v_cache`` are then the same tensor.  ``every``: the mixer keeps one row per
     ``every`` positions (a summary of each whole block of that many): row r belongs to positions r*every .. r*every +
-    every - 1, and the slot that a step names for a token is the row of the token's block; no window."""
+    every - 1, and the slot that a step names for a token is the row of the token's block; no window.  ``keep_first``: beside
+    the window, the sequence's first ``keep_first`` tokens are read for ever (their pages are never given back)."""
 
     num_kv_heads: int
     head_dim: int
@@ -49,6 +50,7 @@ class PagedKVNeed:
     planes: int = 2
     block: int | None = None
     every: int = 1
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

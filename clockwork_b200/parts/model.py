@@ -169,14 +169,22 @@ class DecoderModel:
             self.absolute_positions.add_to_embedding(stream.residual, ctx.positions, self.spec.embedding_scale)
         if self.pair_embedding is not None:
             self.pair_embedding.add_to_embedding(ctx, stream.residual, token_ids, ctx.views[self.pair_cache_layer])
+        input_rows = None
+        if any(step.add_input for step in schedule):
+            input_rows = torch.empty_like(stream.residual).copy_(stream.residual)  # (a device-to-device copy)
         for i, step in enumerate(schedule):
+            if step.add_input:
+                self._add_input(stream, input_rows, self.blocks[step.layer].first_norm())
             view = ctx.views.get(step.resolved_cache_layer())
             if view is not None and hasattr(view, "write"):
                 view.write = step.write_cache
             block = self.blocks[step.layer]
             # the norm that reads the residual next, for blocks that can fuse its first half into their
             # last product (the final norm reads selected rows only and is left alone)
-            following = self.blocks[schedule[i + 1].layer].first_norm() if i + 1 < len(schedule) else None
+            # (input rows added in between come before that norm: a product must not begin it)
+            following = None
+            if i + 1 < len(schedule) and not schedule[i + 1].add_input:
+                following = self.blocks[schedule[i + 1].layer].first_norm()
             if following is not None:
                 block.forward(ctx, stream, view, following_norm=following)
             else:
@@ -186,9 +194,19 @@ class DecoderModel:
             return None
         x = self.final_norm.forward_rows(stream, logit_rows, ctx.status)
         logits = self.head.to_float32(x)
-        if self.spec.logit_softcap is not None:
-            ops.softcap_(logits, self.spec.logit_softcap)
+        if self.spec.logit_softcap is not None or self.spec.logit_scale != 1.0:
+            ops.softcap_(logits, self.spec.logit_softcap, self.spec.logit_scale)
         return logits
+
+    @staticmethod
+    def _add_input(stream: ResidualStream, rows: torch.Tensor, norm) -> None:
+        """``residual += rows`` (float32): inside the kernel of the norm that reads the residual next, when that norm takes
+        slabs and the width suits the kernel that adds them up."""
+        n, w = rows.shape
+        if getattr(norm, "takes_partial_sums", False) and w % 4 == 0 and w <= 4096:
+            stream.push(ops.PartialSums(rows.view(1, n, w), n))
+        else:
+            ops.add_to_residual(stream.residual_after_flush(), rows)
 
 
 def tensor_decls_for_spec(spec: ModelSpec) -> list[TensorDecl]:

@@ -19,7 +19,9 @@ from .base import Norm, ResidualStream
 from .registry import register_norm
 
 
-class RMSNorm(Norm):
+class WeightedNorm(Norm):
+    """What norms of the residual's rows share: a weight [size], an eps, and that the add of what is pending is fused."""
+
     graph_safe = True
     graph_safe_portions = True
     takes_partial_sums = True  # ``forward`` hands whatever the stream holds to ``ops.add_rmsnorm``, slabs included
@@ -41,6 +43,8 @@ class RMSNorm(Norm):
         if self.offset:
             self.weight = (self.weight + self.offset).contiguous()  # float32: exact for a weight stored in bfloat16
 
+
+class RMSNorm(WeightedNorm):
     def split_weight(self) -> torch.Tensor | None:
         """The weight a preceding product multiplies into the residual when it begins this norm."""
         return self.weight if self.dtype == torch.bfloat16 else None

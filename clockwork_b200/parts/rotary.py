@@ -7,15 +7,57 @@ is derived (the reference keeps it out of checkpoints too, ``model.py:169``) and
 
 ``NoPosition`` stores K and V unrotated: the interface another position encoding must have is
 ``apply_and_store(ctx, qkv, view, num_heads, num_kv_heads, head_dim)``.
+
+``rotary_tables`` is what mixers that rotate inside their own kernels make their frequencies with.
 """
 
 from __future__ import annotations
+
+import math
 
 import torch
 
 from .. import ops
 from .base import PagedView, PositionEncoding, StepContext
 from .registry import register_position
+
+
+PAIRINGS = ("half", "interleaved")  # entry i with entry i + dims/2, or entry 2i with entry 2i + 1
+
+
+def check_rotary(rotary: dict, dim: int) -> tuple:
+    """(dims, base, interleaved) of a rotation ``{"dims", "base", "pairing", "scaling"}`` of heads of ``dim`` entries;
+    ``pairing`` is "half" by default, ``scaling`` (absent or None: none) as ``rotary_tables`` takes it."""
+    dims, base, pairing = int(rotary["dims"]), float(rotary["base"]), str(rotary.get("pairing", "half"))
+    if dims <= 0 or dims % 2 or dims > dim or base <= 0:
+        raise ValueError(f"rotary dims {dims} must be even, positive and at most dim {dim}, the base positive")
+    if pairing not in PAIRINGS:
+        raise ValueError(f"rotary pairing must be one of {PAIRINGS}, got {pairing!r}")
+    scaling = rotary.get("scaling")
+    if scaling is not None and (base == 1.0 or min(float(scaling[k]) for k in ("factor", "original", "fast", "slow")) <= 0):
+        raise ValueError("a scaled rotation needs a base other than 1 and positive factor, original, fast and slow")
+    return dims, base, pairing == "interleaved"
+
+
+def rotary_tables(dims: int, base: float, scaling: dict | None = None) -> tuple[torch.Tensor, float]:
+    """(angle per position of every pair, float32 [dims/2]; what sines and cosines are multiplied by).  Worked out in
+    float64 and rounded once.  Plain: ``f_i = base^(-2i/dims)`` and 1.  With ``scaling`` = ``{"factor", "original", "fast",
+    "slow"}`` (YaRN): pairs that turn more than ``fast`` times over ``original`` positions keep their frequency, pairs that
+    turn less than ``slow`` times have it divided by ``factor``, a linear ramp over the pair's index between (its ends
+    rounded outwards to whole indices); sines and cosines are multiplied by ``1 + 0.1 ln(factor)``."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    freq = base ** (-2.0 * i / dims)
+    if scaling is None:
+        return freq.to(torch.float32), 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def index_of(turns: float) -> float:  # of the pair that turns this often over `original` positions
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo = max(math.floor(index_of(float(scaling["fast"]))), 0)
+    hi = min(math.ceil(index_of(float(scaling["slow"]))), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return (freq / factor * ramp + freq * (1.0 - ramp)).to(torch.float32), 0.1 * math.log(factor) + 1.0
 
 
 class RotaryNeox(PositionEncoding):

@@ -39,6 +39,16 @@ dt_bias))`` per head and key channel.  Per head ``S <- diag(a) S; u = beta (v - 
 head's o is divided by its root mean square, times ``norm`` (vdim entries, shared), times ``sigmoid(W_g2 W_g1 x)``, and goes
 through ``o``.  The state slot holds S of every head and the last conv-1 inputs of the convolution.
 
+``head_delta`` (gated delta rule with one decay per head).  Parameters: ``hidden_size, heads, kv_heads, dim, vdim, conv, eps``.
+As ``channel_delta`` with ``g = exp(-exp(A_log[h]) softplus(W_a x + dt_bias))`` per head in the decay's place (``S <- g S``)
+and ``silu(W_g x)`` (heads x vdim) in the gate's; all six products of the input are one.
+
+``retention`` (linear attention with rotary positions and one constant decay per head).  Parameters: ``hidden_size, heads,
+dim, vdim, decay`` (a number per head), ``rotary`` (``rotary.check_rotary``), ``eps``.  The first ``rotary.dims`` entries of every q and
+k head are turned by the token's position (float32 angles), k is multiplied by ``dim^(-1/2)``; per head ``S <- decay_h S +
+k v^T``, ``o = S^T q``.  Each head's o is divided by its root mean square (no weight), times ``silu(W_g x)``, and goes through
+``o``.  The state slot holds S without the factor ``dim^(-1/2)``, which the read-out multiplies by.
+
 ``matrix_memory`` (a matrix memory with exponential gates kept stable by a running maximum).  Parameters: ``hidden_size,
 heads, dim, vdim, gate_cap, eps``.  ``q = W_q x / sqrt(dim)``, ``k, v`` plain products; per head ``li = cap tanh((W_i x +
 b_i)/cap)``, ``lf = log sigmoid(cap tanh((W_f x + b_f)/cap))``, ``m_t = max(lf + m_(t-1), li)`` (m is 0 before the first
@@ -67,6 +77,7 @@ from ..weights.decl import TensorDecl
 from .base import Mixer, ResidualStream, SlotStateNeed, StateView, StepContext
 from .linear import Linear
 from .registry import register_mixer
+from .rotary import check_rotary, rotary_tables
 
 
 class Mamba2Mixer(Mixer):
@@ -278,6 +289,34 @@ class DecayLinearMixer(_LinearAttention):
         return rec_ops.gated_group_norm(o, g, self.norm_w, 1, self.eps, False, self.dtype, gate=rec_ops.GATE_SIGMOID)
 
 
+class RetentionMixer(_LinearAttention):
+    def __init__(self, spec, prefix, dtype, device) -> None:
+        super().__init__(spec, prefix, dtype, device)
+        decay = [float(d) for d in spec["decay"]]
+        if len(decay) != self.heads:
+            raise ValueError(f"decay has {len(decay)} numbers for {self.heads} heads")
+        self.decay = torch.tensor(decay, dtype=torch.float32).to(device)
+        rotary = spec["rotary"]
+        self.rot_dims, base, self.interleaved = check_rotary(rotary, self.dim)
+        inv_freq, self.rot_amplitude = rotary_tables(self.rot_dims, base, rotary.get("scaling"))
+        self.inv_freq = inv_freq.to(device)
+
+    def tensor_decls(self):
+        yield from self._projection_decls()
+
+    def load_weights(self, fetch) -> None:
+        self._load_projections(fetch)
+
+    def _gated_output(self, ctx: StepContext, x, view: StateView):
+        proj = self.w_in.to_float32(x)  # [N, q | k | v | gate], float32
+        rec_ops.rotate_heads_(proj, ctx.positions, self.inv_freq, 2 * self.heads, self.dim, self.rot_dims, self.interleaved,
+                              self.rot_amplitude)
+        q, k, v, g = self._split(proj)
+        o = rec_ops.recurrence_scan(rec_ops.FORM_HEAD_DECAY, q=q, k=k, v=v, pre=None, p0=self.decay, p1=None, p2=None, view=view,
+                                    offset=0, ctx=ctx, heads=self.heads, dk=self.dim, dv=self.vdim, q_scale=self.dim ** -0.5)
+        return rec_ops.gated_group_norm(o, g, None, self.heads, self.eps, False, self.dtype, gate=rec_ops.GATE_SILU)
+
+
 class BoundedForgetMixer(Mixer):
     """``hgrn2``: see the module's text.  One product for ``[q | f | v]`` with float32 output; one kernel makes silu(q), the
     gates f and 1 - f; the scan is the one of ``gated_linear`` with 1 - f in the key's place."""
@@ -331,7 +370,10 @@ class BoundedForgetMixer(Mixer):
         return self.o.add_or_defer(self._normed_output(ctx, x, view), stream)
 
 
-class ChannelDeltaMixer(Mixer):
+class _DeltaRule(Mixer):
+    """What the two delta-rule mixers share: sizes, the state row (S of every head, then the convolutions' last inputs) and
+    the tensors of q, k, v with their convolutions, the write strength, the decay's base and the output."""
+
     graph_safe = True
     graph_safe_portions = True
     UNIT_EPS = 1e-6  # inside the root of the unit vectors' lengths
@@ -343,19 +385,17 @@ class ChannelDeltaMixer(Mixer):
         self.heads, self.kv_heads = int(p["heads"]), int(p["kv_heads"])
         self.dim, self.vdim, self.taps = int(p["dim"]), int(p["vdim"]), int(p["conv"])
         self.eps = float(p["eps"])
-        self.decay_rank, self.gate_rank = int(p.get("decay_rank") or 16), int(p.get("gate_rank") or 16)
         if min(self.heads, self.kv_heads, self.dim, self.vdim, self.taps) <= 0 or self.heads % self.kv_heads:
             raise ValueError(f"heads {self.heads} must be a positive multiple of kv_heads {self.kv_heads}; dim, vdim, conv positive")
         self.qk, self.inner = self.kv_heads * self.dim, self.heads * self.vdim
         self.channels = 2 * self.qk + self.inner       # what passes the convolution: q, k, v
-        self.decays = self.heads * self.dim
         self.scan_offset = 0
         self.conv_offset = self.heads * self.dim * self.vdim
 
     def cache_need(self) -> SlotStateNeed:
         return SlotStateNeed((self.conv_offset + (self.taps - 1) * self.channels,))
 
-    def tensor_decls(self):
+    def _shared_decls(self):
         h = self.hidden_size
         for s, out in (("q", self.qk), ("k", self.qk), ("v", self.inner)):
             yield TensorDecl(self.name(s), (out, h), "matrix", "linear")
@@ -363,24 +403,65 @@ class ChannelDeltaMixer(Mixer):
         yield TensorDecl(self.name("b"), (self.heads, h), "matrix", "linear")
         yield TensorDecl(self.name("A_log"), (self.heads,), "vector", "bias")
         yield TensorDecl(self.name("norm"), (self.vdim,), "vector", "norm")
+        yield TensorDecl(self.name("o"), (h, self.inner), "matrix", "linear")
+
+    def _load_shared(self, fetch, joint) -> None:
+        """``joint``: the tensors whose rows make up the one product of the input."""
+        self.w_in = Linear(torch.cat([fetch(self.name(s)) for s in joint], dim=0).contiguous())
+        self.conv_w = torch.cat([fetch(self.name(f"{s}.conv")) for s in ("q", "k", "v")], dim=0).contiguous()
+        self.a_log, self.dt_bias = fetch(self.name("A_log")).contiguous(), fetch(self.name("dt_bias")).contiguous()
+        self.norm_w = fetch(self.name("norm")).contiguous()
+        self.o = Linear(fetch(self.name("o")))
+
+    def mix(self, ctx: StepContext, x, view: StateView):
+        return self.o.to_float32(self._gated_output(ctx, x, view))
+
+    def forward(self, ctx: StepContext, x, view: StateView, stream: ResidualStream):
+        return self.o.add_or_defer(self._gated_output(ctx, x, view), stream)
+
+
+class HeadDeltaMixer(_DeltaRule):
+    def tensor_decls(self):
+        yield from self._shared_decls()
+        yield TensorDecl(self.name("a"), (self.heads, self.hidden_size), "matrix", "linear")
+        yield TensorDecl(self.name("dt_bias"), (self.heads,), "vector", "bias")
+        yield TensorDecl(self.name("g"), (self.inner, self.hidden_size), "matrix", "linear")
+
+    def load_weights(self, fetch) -> None:
+        self._load_shared(fetch, ("q", "k", "v", "g", "b", "a"))
+
+    def _gated_output(self, ctx: StepContext, x, view: StateView):
+        c, i, h = self.channels, self.inner, self.heads
+        proj = self.w_in.to_float32(x)  # [N, q | k | v | gate | beta | decay], float32
+        o = rec_ops.head_delta(proj, self.conv_w, proj[:, c + i : c + i + h], proj[:, c + i + h :], self.dt_bias, self.a_log, view,
+                               self.scan_offset, self.conv_offset, ctx, self.kv_heads, h, self.dim, self.vdim, self.UNIT_EPS,
+                               self.dim ** -0.5)
+        return rec_ops.gated_group_norm(o, proj[:, c : c + i], self.norm_w, h, self.eps, False, self.dtype, gate=rec_ops.GATE_SILU,
+                                        shared_weight=True)
+
+
+class ChannelDeltaMixer(_DeltaRule):
+    def __init__(self, spec, prefix, dtype, device) -> None:
+        super().__init__(spec, prefix, dtype, device)
+        self.decay_rank, self.gate_rank = int(spec.get("decay_rank") or 16), int(spec.get("gate_rank") or 16)
+        self.decays = self.heads * self.dim
+
+    def tensor_decls(self):
+        h = self.hidden_size
+        yield from self._shared_decls()
         yield TensorDecl(self.name("a1"), (self.decay_rank, h), "matrix", "linear", free_dims=(0,))
         yield TensorDecl(self.name("a2"), (self.decays, self.decay_rank), "matrix", "linear", free_dims=(1,))
         yield TensorDecl(self.name("dt_bias"), (self.decays,), "vector", "bias")
         yield TensorDecl(self.name("g1"), (self.gate_rank, h), "matrix", "linear", free_dims=(0,))
         yield TensorDecl(self.name("g2"), (self.inner, self.gate_rank), "matrix", "linear", free_dims=(1,))
-        yield TensorDecl(self.name("o"), (h, self.inner), "matrix", "linear")
 
     def load_weights(self, fetch) -> None:
-        self.w_in = Linear(torch.cat([fetch(self.name(s)) for s in ("q", "k", "v", "b")], dim=0).contiguous())
-        self.conv_w = torch.cat([fetch(self.name(f"{s}.conv")) for s in ("q", "k", "v")], dim=0).contiguous()
-        self.a_log, self.dt_bias = fetch(self.name("A_log")).contiguous(), fetch(self.name("dt_bias")).contiguous()
-        self.norm_w = fetch(self.name("norm")).contiguous()
+        self._load_shared(fetch, ("q", "k", "v", "b"))
         self.a1, self.a2 = Linear(fetch(self.name("a1"))), Linear(fetch(self.name("a2")))
         self.g1, self.g2 = Linear(fetch(self.name("g1"))), Linear(fetch(self.name("g2")))
         for first, second in ((self.a1, self.a2), (self.g1, self.g2)):
             if first.out_features != second.in_features:
                 raise ValueError(f"{self.prefix}: a product of {first.out_features} rows feeds one of {second.in_features} columns")
-        self.o = Linear(fetch(self.name("o")))
 
     def _gated_output(self, ctx: StepContext, x, view: StateView):
         qk, c = self.qk, self.channels
@@ -396,12 +477,6 @@ class ChannelDeltaMixer(Mixer):
         gate = self.g2.to_float32(self.g1(x))
         return rec_ops.gated_group_norm(o, gate, self.norm_w, self.heads, self.eps, False, self.dtype, gate=rec_ops.GATE_SIGMOID,
                                         shared_weight=True)
-
-    def mix(self, ctx: StepContext, x, view: StateView):
-        return self.o.to_float32(self._gated_output(ctx, x, view))
-
-    def forward(self, ctx: StepContext, x, view: StateView, stream: ResidualStream):
-        return self.o.add_or_defer(self._gated_output(ctx, x, view), stream)
 
 
 class MatrixMemoryMixer(Mixer):
@@ -457,6 +532,8 @@ class MatrixMemoryMixer(Mixer):
 
 register_mixer("hgrn2", BoundedForgetMixer, replace=True)
 register_mixer("channel_delta", ChannelDeltaMixer, replace=True)
+register_mixer("head_delta", HeadDeltaMixer, replace=True)
+register_mixer("retention", RetentionMixer, replace=True)
 register_mixer("matrix_memory", MatrixMemoryMixer, replace=True)
 register_mixer("gated_linear", GatedLinearMixer, replace=True)
 register_mixer("decay_linear", DecayLinearMixer, replace=True)

@@ -22,7 +22,13 @@ Parameters: ``hidden_size, heads, kv_heads, dim`` (query/key size per head), ``v
 * ``query_temperature``: ``{"coef", "every"}``: the query at position t is multiplied by ``1 + coef ln(floor((t + 1) / every) + 1)``;
 * ``gate``: head h's output is multiplied by ``sigmoid(W_g x)_h`` before the output product (tensor ``g`` [heads, hidden]);
 * ``rotary``: ``{"dims", "base"}``: the first ``dims`` entries of every query and key head are rotated by the token's
-  position before the key is cached, entry i with entry i + dims/2 by the angle ``t * base^(-2i/dims)`` (float32).
+  position before the key is cached, entry i with entry i + dims/2 by the angle ``t * base^(-2i/dims)`` (float32);
+  ``"pairing": "interleaved"`` pairs entry 2i with entry 2i + 1 instead, ``"scaling"`` stretches the frequencies
+  (``rotary.rotary_tables``);
+* ``keep_first``: the sequence's first ``keep_first`` positions stay visible (at their own positions) when the window has
+  left them;
+* ``qk_norm``: an eps: before the rotation all of a token's queries together are divided by their root mean square and
+  multiplied by a weight per entry, and all of its keys likewise (tensors ``q.norm`` [heads*dim], ``k.norm`` [kv_heads*dim]).
 
 Without ``rotary`` positions do not enter the scores.  Tensors: ``q`` [heads*dim, hidden], ``k`` [kv_heads*dim, hidden], ``v``
 [kv_heads*vdim, hidden], ``o`` [hidden, heads*vdim], and those the switches name.
@@ -33,7 +39,7 @@ whichever reaches farther back, since a block's mean is taken from the cached ro
 rows live in a page group of one row per ``pool`` positions, ``PagedKVNeed(every=pool)``).  At load the rows of k and v are
 interleaved head by head behind q, so that one product yields ``[q | k_0 v_0 | k_1 v_1 ..]`` per token and the
 cache write is a copy of the row's tail (with ``rotary`` the product's output is float32 and one kernel rotates,
-rounds once and stores).  A blocked layer's page group gives back the pages of blocks that have passed.
+(and norms) rounds once and stores).  A blocked layer's page group gives back the pages of blocks that have passed.
 Scores, weights and weighted sums are float32 in either run precision.
 """
 
@@ -46,6 +52,7 @@ from ..weights.decl import TensorDecl
 from .base import Mixer, PagedKVNeed, PagedView, ResidualStream, StepContext
 from .linear import Linear
 from .registry import register_mixer
+from .rotary import check_rotary, rotary_tables
 
 
 class WindowAttention(Mixer):
@@ -89,12 +96,16 @@ class WindowAttention(Mixer):
             raise ValueError("query_temperature.every must be at least 1")
         self.has_gate = bool(p.get("gate", False))
         self.slopes = None
-        rotary = p.get("rotary")
-        self.rot_dims = int(rotary["dims"]) if rotary else 0
-        self.rot_base = float(rotary["base"]) if rotary else 0.0
-        if rotary and (self.rot_dims <= 0 or self.rot_dims % 2 or self.rot_dims > int(p["dim"]) or self.rot_base <= 0):
-            raise ValueError(f"rotary dims {self.rot_dims} must be even, positive and at most dim {p['dim']}, the base positive")
-        self.inv_freq = self.sink = None
+        self.keep_first = int(p.get("keep_first") or 0)
+        if self.window >= window_ops.NO_WINDOW:
+            self.keep_first = 0  # (a window that never closes leaves nothing)
+        if self.keep_first < 0 or (self.keep_first and (self.mask != "window" or self.pool)):
+            raise ValueError("kept first positions lie before a sliding window without pooled blocks")
+        self.qk_eps = None if p.get("qk_norm") is None else float(p["qk_norm"])
+        self.rotary = p.get("rotary")
+        self.rot_dims, self.rot_base, self.interleaved = check_rotary(self.rotary, self.dim) if self.rotary else (0, 0.0, False)
+        self.rot_amplitude = 1.0
+        self.inv_freq = self.sink = self.q_norm = self.k_norm = None
         if self.heads <= 0 or self.kv_heads <= 0 or self.heads % self.kv_heads:
             raise ValueError(f"heads {self.heads} not a multiple of kv_heads {self.kv_heads}")
         if min(self.dim, self.vdim, self.window) <= 0:
@@ -113,7 +124,7 @@ class WindowAttention(Mixer):
             # (a block's mean is read from the cached rows when its last token arrives: the last `pool` positions stay too)
             return (PagedKVNeed(self.kv_heads, self.row, max(self.window, self.pool), planes=1),
                     PagedKVNeed(self.kv_heads, self.row, None, planes=1, every=self.pool))
-        return PagedKVNeed(self.kv_heads, self.row, self.window, planes=1)
+        return PagedKVNeed(self.kv_heads, self.row, self.window, planes=1, keep_first=self.keep_first)
 
     def reserve_for_steps(self, max_seqs: int, max_ctx: int) -> None:
         if self.device.type == "cuda":
@@ -125,6 +136,9 @@ class WindowAttention(Mixer):
             yield TensorDecl(self.name(name), (out, h), "matrix", "linear")
             if self.bias:
                 yield TensorDecl(self.name(f"{name}.b"), (out,), "vector", "bias")
+        if self.qk_eps is not None:
+            yield TensorDecl(self.name("q.norm"), (self.heads * self.dim,), "vector", "norm")
+            yield TensorDecl(self.name("k.norm"), (self.kv_heads * self.dim,), "vector", "norm")
         if self.has_head_scale:
             yield TensorDecl(self.name("temp"), (self.heads,), "vector", "norm")
         if self.has_talk:
@@ -168,21 +182,24 @@ class WindowAttention(Mixer):
         if self.halvings:
             h = torch.arange(1, self.heads + 1, dtype=torch.float64)
             self.slopes = torch.pow(2.0, -self.halvings * h / self.heads).to(torch.float32).to(w.device)
+        if self.qk_eps is not None:
+            self.q_norm, self.k_norm = (fetch(self.name(f"{n}.norm")).contiguous() for n in "qk")
         if self.rot_dims:
-            # base^(-2i/dims) worked out in float64 and rounded once
-            i = torch.arange(self.rot_dims // 2, dtype=torch.float64)
-            self.inv_freq = (self.rot_base ** (-2.0 * i / self.rot_dims)).to(torch.float32).to(self.qkv.weight.device)
+            inv_freq, self.rot_amplitude = rotary_tables(self.rot_dims, self.rot_base, self.rotary.get("scaling"))
+            self.inv_freq = inv_freq.to(self.qkv.weight.device)
 
     def _attend(self, ctx: StepContext, x: torch.Tensor, view) -> torch.Tensor:
         view, pooled = view if self.pool else (view, None)
         rows = view.k_cache  # [pages, page_size, kv_heads, dim + vdim]
         gate = None
-        if self.rot_dims or self.has_gate:
+        if self.rot_dims or self.has_gate or self.qk_eps is not None:
             # the product in float32, so that rotated queries and keys are rounded to the run's precision once (and the
             # gate's logits not at all)
             proj = self.qkv.to_float32(x)
             q = window_ops.rotate_store(proj, ctx.positions, ctx.tok_seq, view.slots if view.write else None,
-                                        self.inv_freq, self.heads, self.kv_heads, self.dim, self.vdim, self.rot_dims, rows, ctx.status)
+                                        self.inv_freq, self.heads, self.kv_heads, self.dim, self.vdim, self.rot_dims, rows, ctx.status,
+                                        self.interleaved, self.rot_amplitude,
+                                        None if self.qk_eps is None else (self.q_norm, self.k_norm, self.qk_eps))
             if self.has_gate:
                 gate = proj[:, self.heads * self.dim + self.kv_heads * self.row :]
         else:
@@ -198,7 +215,7 @@ class WindowAttention(Mixer):
                                            blocked=self.mask == "block", sink=self.sink, softcap=self.softcap, slopes=self.slopes,
                                            temperature=self.temperature, gate=gate, pool=self.pool,
                                            pool_rows_cache=pooled.k_cache if self.pool else None,
-                                           pool_tables=pooled.block_tables if self.pool else None)
+                                           pool_tables=pooled.block_tables if self.pool else None, keep_first=self.keep_first)
 
     def mix(self, ctx: StepContext, x: torch.Tensor, view: PagedView) -> torch.Tensor:
         return self.o.to_float32(self._attend(ctx, x, view))
