@@ -379,7 +379,10 @@ def compare_designs(args) -> int:
     64 pooled before it, a recurrent layer with bounded forget gates in every fourth place, 32 routed experts of which a
     token uses 4, 7,168 feed-forward rows a token, a hashed pair table and the average over the depth) beside Kapolorn, the
     closest design the framework has (``kapolorn-2k``: the same width, heads and layer count, the same attention and
-    expert kernels).  With ``--layers N`` both models have N layers.  One JSON
+    expert kernels).  With ``--design dezolorn`` the design is Dezolorn (``dezolorn-2k``: attention over a window of 1,024
+    positions and the first 4, retention and delta-rule layers of 16 heads of 128 x 128, gated feed-forwards of 7,168, an output
+    head of its own) beside Gamesun, the closest design the framework has (``gamesun-2k``: the same width, heads, layer
+    count and feed-forward; its layers run two mixers each, Dezolorn's one).  With ``--layers N`` both models have N layers.  One JSON
     line; device time by CUDA events, medians."""
     import torch
 
@@ -389,7 +392,8 @@ def compare_designs(args) -> int:
 
     assert torch.cuda.is_available(), "bench.py needs a CUDA device"
     torch.cuda.set_device(0)
-    shape = {"rapitar": "rapitar-2k", "gamesun": "gamesun-2k", "kapolorn": "kapolorn-2k", "nuzulorn": "nuzulorn-2k"}[args.design]
+    shape = {"rapitar": "rapitar-2k", "gamesun": "gamesun-2k", "kapolorn": "kapolorn-2k", "nuzulorn": "nuzulorn-2k",
+             "dezolorn": "dezolorn-2k"}[args.design]
     rapitar = shape_config(shape, args.layers)
     layers = len(rapitar["layers"])
     qwen = dict(QWEN25_1P5B, num_hidden_layers=layers, hidden_size=2048, num_attention_heads=16,
@@ -399,7 +403,7 @@ def compare_designs(args) -> int:
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda:0")  # larger than L2: written between timed calls
     out = {"impl": "ours", "layers": layers, "width": 2048, "dtype": "bf16", "data": "synthetic", "l2": "flushed between timed calls"}
     beside = ("qwen2-2k", qwen, qwen["vocab_size"])
-    if args.design == "kapolorn":
+    if args.design in ("kapolorn", "dezolorn"):
         beside = ("gamesun-2k", shape_config("gamesun-2k", layers), rapitar["vocab"])
     if args.design == "nuzulorn":
         beside = ("kapolorn-2k", shape_config("kapolorn-2k", layers), rapitar["vocab"])
@@ -470,7 +474,7 @@ def main() -> int:
     ap.add_argument("--top-k", type=int, default=-1)
     ap.add_argument("--top-p", type=float, default=1.0)
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the shape has (reported in config)")
-    ap.add_argument("--design", choices=["rapitar", "gamesun", "kapolorn", "nuzulorn"], default="rapitar", help="with --only designs: which design stands beside Qwen2")
+    ap.add_argument("--design", choices=["rapitar", "gamesun", "kapolorn", "nuzulorn", "dezolorn"], default="rapitar", help="with --only designs: which design stands beside Qwen2")
     ap.add_argument("--model-filter", default="", help="with --only designs: run only the model whose name holds this text (profiling runs)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--shape", default="qwen2.5-1.5b",

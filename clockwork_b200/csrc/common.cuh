@@ -68,6 +68,34 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// part[0 .. TOKENS-1] of each of IP neighbouring lanes (lane `ipart` of its group; IP a power of two): every token's sum over
+// the lanes, with the tokens spread over the lanes while they are summed: a lane keeps one half of the tokens it holds and
+// hands the other half on.  Returns the first token whose sum this lane ends up with (its TOKENS / IP tokens, at least one, are
+// in part[0 ..]), or -1 for a lane whose sum another lane holds too.  The order of a token's sum depends on IP alone.
+template <int IP, int TOKENS>
+__device__ __forceinline__ int sum_tokens_over_lanes(float (&part)[TOKENS], int ipart) {
+    int held = TOKENS, first = 0;
+#pragma unroll
+    for (int o = IP >> 1; o >= 1; o >>= 1) {
+        if (held > 1) {
+            held >>= 1;
+            const bool upper = (ipart & o) != 0;
+#pragma unroll
+            for (int i = 0; i < TOKENS / 2; ++i)
+                if (i < held) {
+                    const float send = upper ? part[i] : part[i + held];
+                    const float keep = upper ? part[i + held] : part[i];
+                    part[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+                }
+            if (upper) first += held;
+        } else {
+            part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
+            if (ipart & o) first = -1;
+        }
+    }
+    return first;
+}
+
 // Block-wide reductions with a fixed order (warp tree, then warp 0 over the warp results),
 // so the result for a row never depends on what else is in the batch.
 // `scratch` must hold 33 floats.  All threads receive the result.

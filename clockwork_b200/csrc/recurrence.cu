@@ -199,17 +199,23 @@ __device__ __forceinline__ void cp_async4(float* smem, const float* gmem) {
 // current one is computed) and read from there by the IP x JB threads; a thread owns key channels ipart, ipart + IP, ..
 // of value column j, so that neighbouring lanes read neighbouring words of shared memory and of the state.
 // The per-token sums over key channels are reduced over the IP lanes of a column after the chunk's loop.
-template <int FORM, bool VEC>
+// IPT > 0: IP known at compile time, heads of whole groups of eight channels at 16-byte addresses (lanes beyond Dk / 8 own no
+// channels), and the chunk's tokens spread over the lanes while their sums are formed (sum_tokens_over_lanes); 0: any head size.
+template <int FORM, int IPT>
 __global__ void __launch_bounds__(256)
 recurrence_scan_kernel(const float* __restrict__ q, int ldq, const float* __restrict__ k, int ldk,
                        const float* __restrict__ v, int ldv, const float* __restrict__ pre, int ldp,
                        const float* __restrict__ p0, const float* __restrict__ p1, const float* __restrict__ p2,
                        float* __restrict__ state, long long state_stride, long long state_off,
                        const long long* __restrict__ slots, const int* __restrict__ tok_seq,
-                       const int* __restrict__ q_start, int Dk, int Dv, int heads_per_group, int IP, int wide, int H,
+                       const int* __restrict__ q_start, int Dk, int Dv, int heads_per_group, int ip, int wide, int H,
                        float* __restrict__ out, int ldo, float q_scale) {
     extern __shared__ __align__(16) float rs_smem[];
+    __shared__ __align__(16) float nothing[4];  // zeros: what lanes without channels read
+    if (threadIdx.x < 4) nothing[threadIdx.x] = 0.f;
     pdl_wait();
+    constexpr bool VEC = IPT > 0;
+    const int IP = VEC ? IPT : ip;
     const int seq = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int start = q_start[seq], end = q_start[seq + 1];
     if (end <= start) return;
@@ -228,16 +234,18 @@ recurrence_scan_kernel(const float* __restrict__ q, int ldq, const float* __rest
     const int buf_words = 2 * RC * Dk + a_words + RC * JB;
     const int g = h / heads_per_group;
     float* S_mem = state + slots[seq] * state_stride + state_off + ((size_t)h * Dv + (live ? j : 0)) * Dk;
-    // VEC (Dk == 8 IP): a thread owns channels 4 ipart .. 4 ipart + 3 and the same four in the upper half, read as
+    // VEC: a thread owns channels 4 ipart .. 4 ipart + 3 and the same four in the upper half, read as
     // two 16-byte words per operand and token (neighbouring lanes read neighbouring words: no bank conflicts);
     // otherwise channels ipart, ipart + IP, .. one word at a time
     const int half = Dk >> 1;
+    const bool mine = ipart * RS < Dk;  // (VEC: the thread owns channels at all)
+    const int token_step = mine ? Dk : 0, upper = mine ? half : 0;
     auto channel = [&](int r) { return VEC ? (r < 4 ? 0 : half) + ipart * 4 + (r & 3) : ipart + r * IP; };
     float S[RS], c1[RS];
 #pragma unroll
     for (int r = 0; r < RS; ++r) {
         const int i = channel(r);
-        const bool on = i < Dk;
+        const bool on = VEC ? mine : i < Dk;
         S[r] = (on && live) ? S_mem[i] : 0.f;
         if (FORM == 0) c1[r] = on ? p1[(size_t)h * Dk + i] : 0.f;
     }
@@ -257,9 +265,8 @@ recurrence_scan_kernel(const float* __restrict__ q, int ldq, const float* __rest
         float* vs = as + a_words;
         if (wide) {  // rows of whole 16-byte pieces at 16-byte addresses
             const int pieces = Dk >> 2;
-            const int shift = VEC ? 31 - __clz(pieces) : 0;  // (VEC: Dk = 8 * 2^n, so a power of two)
             for (int idx = tid; idx < n * pieces; idx += blockDim.x) {
-                const int t = VEC ? idx >> shift : idx / pieces, i = (idx - t * pieces) << 2;
+                const int t = idx / pieces, i = (idx - t * pieces) << 2;
                 cp_async16f(qs + t * Dk + i, qp + (size_t)(t0 + t) * ldq + i);
                 cp_async16f(ks + t * Dk + i, kp + (size_t)(t0 + t) * ldk + i);
                 if (CH) cp_async16f(as + t * Dk + i, pp + (size_t)(t0 + t) * ldp + i);
@@ -295,75 +302,92 @@ recurrence_scan_kernel(const float* __restrict__ q, int ldq, const float* __rest
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();  // this chunk has landed; everyone has left the other buffer
         if (t0 + RC < end) fetch(t0 + RC, rs_smem + (which ^ 1) * buf_words);
-        float part[RC];
+        const float* q0 = mine ? qs + ipart * 4 : nothing;
+        const float* k0 = mine ? ks + ipart * 4 : nothing;
+        const float* a0 = mine ? as + ipart * 4 : nothing;
+        auto token = [&](int t) {  // the thread's share of token t's output; its columns of the state move on by the token
+            const float vraw = live ? ((FORM == 4 && j == Dv - 1) ? 1.f : vs[t * JB + jl]) : 0.f;
+            const float a1 = HD ? as[t] : head_decay;
+            const float vc = HD ? vraw * as[RC + t] : vraw;  // the step size scales the update
+            float sum = 0.f;
+            if (VEC) {
+                const int at = t * token_step;
+                float kc[RS], qc[RS], ac[RS];
+                *(float4*)&kc[0] = *(const float4*)(k0 + at);
+                *(float4*)&kc[4] = *(const float4*)(k0 + at + upper);
+                *(float4*)&qc[0] = *(const float4*)(q0 + at);
+                *(float4*)&qc[4] = *(const float4*)(q0 + at + upper);
+                if (CH) {
+                    *(float4*)&ac[0] = *(const float4*)(a0 + at);
+                    *(float4*)&ac[4] = *(const float4*)(a0 + at + upper);
+                }
+                float sum2 = 0.f;  // two chains of four, added at the end: the same order for every token and batch
 #pragma unroll
-        for (int t = 0; t < RC; ++t) {
-            part[t] = 0.f;
-            if (t < n) {
-                const float vraw = live ? ((FORM == 4 && j == Dv - 1) ? 1.f : vs[t * JB + jl]) : 0.f;
-                const float a1 = HD ? as[t] : head_decay;
-                const float vc = HD ? vraw * as[RC + t] : vraw;  // the step size scales the update
-                float sum = 0.f;
-                if (VEC) {
-                    const int at = t * Dk + ipart * 4, up = at + half;
-                    float kc[RS], qc[RS], ac[RS];
-                    *(float4*)&kc[0] = *(const float4*)(ks + at);
-                    *(float4*)&kc[4] = *(const float4*)(ks + up);
-                    *(float4*)&qc[0] = *(const float4*)(qs + at);
-                    *(float4*)&qc[4] = *(const float4*)(qs + up);
-                    if (CH) {
-                        *(float4*)&ac[0] = *(const float4*)(as + at);
-                        *(float4*)&ac[4] = *(const float4*)(as + up);
+                for (int r = 0; r < RS; ++r) {
+                    const float kv = kc[r] * vc;
+                    float& acc_sum = r < 4 ? sum : sum2;
+                    if (FORM == 0) {
+                        acc_sum = fmaf(qc[r], fmaf(c1[r], kv, S[r]), acc_sum);
+                        S[r] = fmaf(ac[r], S[r], kv);
+                    } else {
+                        S[r] = fmaf(CH ? ac[r] : a1, S[r], kv);
+                        acc_sum = fmaf(qc[r], S[r], acc_sum);
                     }
-                    float sum2 = 0.f;  // two chains of four, added at the end: the same order for every token and batch
+                }
+                sum += sum2;
+            } else {
 #pragma unroll
-                    for (int r = 0; r < RS; ++r) {
-                        const float kv = kc[r] * vc;
-                        float& acc_sum = r < 4 ? sum : sum2;
+                for (int r = 0; r < RS; ++r) {
+                    const int i = ipart + r * IP;
+                    if (i < Dk) {
+                        const float kv = ks[t * Dk + i] * vc, qc = qs[t * Dk + i];
                         if (FORM == 0) {
-                            acc_sum = fmaf(qc[r], fmaf(c1[r], kv, S[r]), acc_sum);
-                            S[r] = fmaf(ac[r], S[r], kv);
+                            sum = fmaf(qc, fmaf(c1[r], kv, S[r]), sum);
+                            S[r] = fmaf(as[t * Dk + i], S[r], kv);
                         } else {
-                            S[r] = fmaf(CH ? ac[r] : a1, S[r], kv);
-                            acc_sum = fmaf(qc[r], S[r], acc_sum);
-                        }
-                    }
-                    sum += sum2;
-                } else {
-#pragma unroll
-                    for (int r = 0; r < RS; ++r) {
-                        const int i = ipart + r * IP;
-                        if (i < Dk) {
-                            const float kv = ks[t * Dk + i] * vc, qc = qs[t * Dk + i];
-                            if (FORM == 0) {
-                                sum = fmaf(qc, fmaf(c1[r], kv, S[r]), sum);
-                                S[r] = fmaf(as[t * Dk + i], S[r], kv);
-                            } else {
-                                S[r] = fmaf(CH ? as[t * Dk + i] : a1, S[r], kv);
-                                sum = fmaf(qc, S[r], sum);
-                            }
+                            S[r] = fmaf(CH ? as[t * Dk + i] : a1, S[r], kv);
+                            sum = fmaf(qc, S[r], sum);
                         }
                     }
                 }
-                part[t] = sum;
             }
-        }
+            return sum;
+        };
+        float part[RC];
+        if (n == RC) {
 #pragma unroll
-        for (int t = 0; t < RC; ++t)
-            for (int o = 1; o < IP; o <<= 1) part[t] += __shfl_xor_sync(0xffffffffu, part[t], o);
-        if (live && ipart == 0) {
+            for (int t = 0; t < RC; ++t) part[t] = token(t);
+        } else {
+#pragma unroll
+            for (int t = 0; t < RC; ++t) part[t] = t < n ? token(t) : 0.f;
+        }
+        auto write = [&](int t, float y) {
+            out[(size_t)(t0 + t) * ldo + (size_t)h * Dv + j] =
+                FORM == 1 ? fmaf(head_skip, vs[t * JB + jl], y) : (FORM >= 2 ? y * q_scale : y);
+        };
+        if (VEC) {
+            const int first = sum_tokens_over_lanes<VEC ? IPT : 1, RC>(part, ipart);
+            if (live && first >= 0) {
+#pragma unroll
+                for (int i = 0; i < (IPT > RC ? 1 : RC / (VEC ? IPT : 1)); ++i)
+                    if (first + i < n) write(first + i, part[i]);
+            }
+        } else {
 #pragma unroll
             for (int t = 0; t < RC; ++t)
-                if (t < n)
-                    out[(size_t)(t0 + t) * ldo + (size_t)h * Dv + j] =
-                        FORM == 1 ? fmaf(head_skip, vs[t * JB + jl], part[t]) : (FORM >= 2 ? part[t] * q_scale : part[t]);
+                for (int o = 1; o < IP; o <<= 1) part[t] += __shfl_xor_sync(0xffffffffu, part[t], o);
+            if (live && ipart == 0) {
+#pragma unroll
+                for (int t = 0; t < RC; ++t)
+                    if (t < n) write(t, part[t]);
+            }
         }
     }
     if (live) {
 #pragma unroll
         for (int r = 0; r < RS; ++r) {
             const int i = channel(r);
-            if (i < Dk) S_mem[i] = S[r];
+            if (VEC ? mine : i < Dk) S_mem[i] = S[r];
         }
     }
 }
@@ -377,8 +401,11 @@ extern "C" int cw_recurrence_scan(int form, const float* q, int ldq, const float
     if (S == 0) return CW_OK;
     if (S < 0 || H <= 0 || Dk <= 0 || Dv <= 0 || heads_per_group <= 0 || H % heads_per_group) return CW_ERR_BAD_SIZE;
     if (Dk > 32 * RS || H > 65535) return CW_ERR_UNSUPPORTED;
-    int IP = 1;
-    while (IP * RS < Dk) IP *= 2;
+    int IP = 1, log_ip = 0;
+    while (IP * RS < Dk) {
+        IP *= 2;
+        ++log_ip;
+    }
     int threads = 256;  // more value columns per block share the staged q and k; fewer when a head has few columns
     while (threads > 32 && threads / IP >= 2 * Dv) threads /= 2;
     const int JB = threads / IP;
@@ -390,22 +417,22 @@ extern "C" int cw_recurrence_scan(int form, const float* q, int ldq, const float
     const int wide = Dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && (!ch || ldp % 4 == 0) && ((uintptr_t)q & 15) == 0 &&
                      ((uintptr_t)k & 15) == 0 && (!ch || ((uintptr_t)pre & 15) == 0);
     const size_t smem = 2 * sizeof(float) * (size_t)(2 * RC * Dk + (ch ? RC * Dk : (form == 1 || form == 4 ? 2 * RC : 0)) + RC * JB);
-    const bool vec = wide && Dk == IP * RS;
-    const int which = form * 2 + (vec ? 1 : 0);
-    static size_t allowed[10] = {48 << 10, 48 << 10, 48 << 10, 48 << 10, 48 << 10, 48 << 10, 48 << 10, 48 << 10, 48 << 10, 48 << 10};
+    const int which = wide && Dk % RS == 0 ? log_ip : 6;
+    static size_t allowed[5][7] = {};
     using Kernel = void (*)(const float*, int, const float*, int, const float*, int, const float*, int, const float*, const float*,
                             const float*, float*, long long, long long, const long long*, const int*, const int*, int, int, int, int, int, int,
                             float*, int, float);
-    const Kernel kernels[10] = {recurrence_scan_kernel<0, false>, recurrence_scan_kernel<0, true>, recurrence_scan_kernel<1, false>,
-                                recurrence_scan_kernel<1, true>, recurrence_scan_kernel<2, false>, recurrence_scan_kernel<2, true>,
-                                recurrence_scan_kernel<3, false>, recurrence_scan_kernel<3, true>, recurrence_scan_kernel<4, false>,
-                                recurrence_scan_kernel<4, true>};
-    if (smem > allowed[which]) {
-        const cudaError_t e = cudaFuncSetAttribute(kernels[which], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+#define CW_FORM(f)                                                                                                              \
+    {recurrence_scan_kernel<f, 1>, recurrence_scan_kernel<f, 2>, recurrence_scan_kernel<f, 4>, recurrence_scan_kernel<f, 8>,     \
+     recurrence_scan_kernel<f, 16>, recurrence_scan_kernel<f, 32>, recurrence_scan_kernel<f, 0>}
+    static const Kernel kernels[5][7] = {CW_FORM(0), CW_FORM(1), CW_FORM(2), CW_FORM(3), CW_FORM(4)};
+#undef CW_FORM
+    if (smem > (48u << 10) && smem > allowed[form][which]) {
+        const cudaError_t e = cudaFuncSetAttribute(kernels[form][which], cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
-        allowed[which] = smem;
+        allowed[form][which] = smem;
     }
-    return cw_launch_ordered(kernels[which], grid, dim3(threads), smem, stream, q, ldq, k, ldk, v, ldv, pre, ldp, p0, p1, p2, state,
+    return cw_launch_ordered(kernels[form][which], grid, dim3(threads), smem, stream, q, ldq, k, ldk, v, ldv, pre, ldp, p0, p1, p2, state,
                      state_stride, state_off, slots, tok_seq, q_start, Dk, Dv, heads_per_group, IP, wide, H, out, ldo, q_scale);
 }
 

@@ -80,61 +80,121 @@ extern "C" int cw_delta_coefficients(float* pre, int ldp, const float* dt_bias, 
 // that pass a causal convolution of `taps` taps per channel (weight [C, taps], the current token's last; inputs before a
 // portion's first row are the rows kept in the request's state) and SiLU; then every q and k head is divided by
 // sqrt(sum of squares + eps), q heads times q_scale.  out [N, C].  beta [N, ldb] and decay [N, lda] hold the pre-activations of a
-// number per head: coef [N, 2H] = [exp(-exp(A[h]) softplus(decay + dt[h])) | sigmoid(beta)].  A block per token; a warp per q or
-// k head, its channels in registers between the sum and the division.
+// number per head: coef [N, 2H] = [exp(-exp(A[h]) softplus(decay + dt[h])) | sigmoid(beta)].  Blocks: (token, share of its heads
+// and channels); a warp per q or k head, its channels in registers between the sum and the division.  VEC: four taps, four
+// neighbouring channels a lane in 16-byte accesses (heads of a multiple of four channels at 16-byte addresses).
 #define DP_CH 8  // channels of a head per lane (heads up to 256 wide)
+struct DeltaPrepareArgs {
+    const float* x;
+    int ldx;
+    const float* weight;
+    int taps;
+    const float* state;
+    long long state_stride, conv_off;
+    const long long* slots;
+    const int* tok_seq;
+    const int* q_start;
+    int groups, Dk, H, Dv;
+    float eps, q_scale;
+    const float* beta;
+    int ldb;
+    const float* decay;
+    int lda;
+    const float* dt_bias;
+    const float* a_log;
+    float* out;
+    float* coef;
+};
+
+template <bool VEC>
 __global__ void __launch_bounds__(256)
-delta_prepare_kernel(const float* __restrict__ x, int ldx, const float* __restrict__ weight, int taps,
-                     const float* __restrict__ state, long long state_stride, long long conv_off, const long long* __restrict__ slots,
-                     const int* __restrict__ tok_seq, const int* __restrict__ q_start, int groups, int Dk, int H, int Dv, float eps,
-                     float q_scale, const float* __restrict__ beta, int ldb, const float* __restrict__ decay, int lda,
-                     const float* __restrict__ dt_bias, const float* __restrict__ a_log, float* __restrict__ out,
-                     float* __restrict__ coef) {
+delta_prepare_kernel(const DeltaPrepareArgs a) {
     pdl_wait();
-    const int row = blockIdx.x, tid = threadIdx.x;
-    const int qk = groups * Dk, C = 2 * qk + H * Dv, R = taps - 1;
-    float* o = out + (size_t)row * C;
-    float* cf = coef + (size_t)row * 2 * H;
-    const int seq = tok_seq[row];
+    const int row = blockIdx.x, tid = threadIdx.x, share = blockIdx.y, shares = gridDim.y;
+    const int Dk = a.Dk, qk = a.groups * Dk, C = 2 * qk + a.H * a.Dv, R = a.taps - 1;
+    const int at = share * blockDim.x + tid, step = shares * blockDim.x;  // this thread's first channel (or four) and the stride
+    float* o = a.out + (size_t)row * C;
+    float* cf = a.coef + (size_t)row * 2 * a.H;
+    const int seq = a.tok_seq[row];
     if (seq < 0) {  // padding of a fixed-shape step
-        for (int c = tid; c < C; c += blockDim.x) o[c] = 0.f;
-        for (int h = tid; h < 2 * H; h += blockDim.x) cf[h] = 0.f;
+        for (int c = at; c < C; c += step) o[c] = 0.f;
+        for (int h = at; h < 2 * a.H; h += step) cf[h] = 0.f;
         return;
     }
-    const int start = q_start[seq];
-    const float* kept = state + slots[seq] * state_stride + conv_off;
+    const int start = a.q_start[seq];
+    const float* kept = a.state + a.slots[seq] * a.state_stride + a.conv_off;
+    auto source = [&](int j) {  // the row that tap j reads
+        const int src = row - (R - j);
+        return src >= start ? a.x + (size_t)src * a.ldx : kept + (size_t)(R - (start - src)) * C;
+    };
+    auto silu = [](float z) { return z / (1.f + expf(-z)); };
     auto conv = [&](int c) {
         float acc = 0.f;
-        for (int j = 0; j < taps; ++j) {
-            const int src = row - (R - j);
-            const float v = src >= start ? x[(size_t)src * ldx + c] : kept[(size_t)(R - (start - src)) * C + c];
-            acc = fmaf(weight[(size_t)c * taps + j], v, acc);
-        }
-        return acc / (1.f + expf(-acc));
+        for (int j = 0; j < a.taps; ++j) acc = fmaf(a.weight[(size_t)c * a.taps + j], source(j)[c], acc);
+        return silu(acc);
     };
-    const int warp = tid >> 5, lane = tid & 31, nwarps = blockDim.x >> 5;
-    for (int head = warp; head < 2 * groups; head += nwarps) {
-        float u[DP_CH], ss = 0.f;
+    const float* rows4[4];
+    if (VEC) {
 #pragma unroll
-        for (int r = 0; r < DP_CH; ++r) {
-            const int i = lane + 32 * r;
-            u[r] = i < Dk ? conv(head * Dk + i) : 0.f;
-            ss = fmaf(u[r], u[r], ss);
-        }
-        ss = warp_sum(ss);
-        const float f = (head < groups ? q_scale : 1.f) / sqrtf(ss + eps);
+        for (int j = 0; j < 4; ++j) rows4[j] = source(j);
+    }
+    auto conv4 = [&](int c) {  // channels c .. c + 3
+        float4 x[4], w[4];
 #pragma unroll
-        for (int r = 0; r < DP_CH; ++r) {
-            const int i = lane + 32 * r;
-            if (i < Dk) o[head * Dk + i] = u[r] * f;
+        for (int j = 0; j < 4; ++j) x[j] = *(const float4*)(rows4[j] + c);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) w[i] = *(const float4*)(a.weight + (size_t)(c + i) * 4);
+        float4 y;
+        y.x = silu(fmaf(w[0].w, x[3].x, fmaf(w[0].z, x[2].x, fmaf(w[0].y, x[1].x, w[0].x * x[0].x))));
+        y.y = silu(fmaf(w[1].w, x[3].y, fmaf(w[1].z, x[2].y, fmaf(w[1].y, x[1].y, w[1].x * x[0].y))));
+        y.z = silu(fmaf(w[2].w, x[3].z, fmaf(w[2].z, x[2].z, fmaf(w[2].y, x[1].z, w[2].x * x[0].z))));
+        y.w = silu(fmaf(w[3].w, x[3].w, fmaf(w[3].z, x[2].w, fmaf(w[3].y, x[1].w, w[3].x * x[0].w))));
+        return y;
+    };
+    const int lane = tid & 31, nwarps = blockDim.x >> 5;
+    for (int head = share * nwarps + (tid >> 5); head < 2 * a.groups; head += shares * nwarps) {
+        float ss = 0.f;
+        const float scale = head < a.groups ? a.q_scale : 1.f;
+        if (VEC) {
+            float4 u[DP_CH / 4];
+#pragma unroll
+            for (int r = 0; r < DP_CH / 4; ++r) {
+                const int i = (lane + 32 * r) * 4;
+                u[r] = i < Dk ? conv4(head * Dk + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+                ss = fmaf(u[r].x, u[r].x, fmaf(u[r].y, u[r].y, fmaf(u[r].z, u[r].z, fmaf(u[r].w, u[r].w, ss))));
+            }
+            const float f = scale / sqrtf(warp_sum(ss) + a.eps);
+#pragma unroll
+            for (int r = 0; r < DP_CH / 4; ++r) {
+                const int i = (lane + 32 * r) * 4;
+                if (i < Dk) *(float4*)(o + head * Dk + i) = make_float4(u[r].x * f, u[r].y * f, u[r].z * f, u[r].w * f);
+            }
+        } else {
+            float u[DP_CH];
+#pragma unroll
+            for (int r = 0; r < DP_CH; ++r) {
+                const int i = lane + 32 * r;
+                u[r] = i < Dk ? conv(head * Dk + i) : 0.f;
+                ss = fmaf(u[r], u[r], ss);
+            }
+            const float f = scale / sqrtf(warp_sum(ss) + a.eps);
+#pragma unroll
+            for (int r = 0; r < DP_CH; ++r) {
+                const int i = lane + 32 * r;
+                if (i < Dk) o[head * Dk + i] = u[r] * f;
+            }
         }
     }
-    for (int c = 2 * qk + tid; c < C; c += blockDim.x) o[c] = conv(c);
-    for (int h = tid; h < H; h += blockDim.x) {
-        const float z = decay[(size_t)row * lda + h] + dt_bias[h];
-        const float step = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
-        cf[h] = expf(-expf(a_log[h]) * step);
-        cf[H + h] = 1.f / (1.f + expf(-beta[(size_t)row * ldb + h]));
+    if (VEC) {
+        for (int c = 2 * qk + 4 * at; c < C; c += 4 * step) *(float4*)(o + c) = conv4(c);
+    } else {
+        for (int c = 2 * qk + at; c < C; c += step) o[c] = conv(c);
+    }
+    for (int h = at; h < a.H; h += step) {
+        const float z = a.decay[(size_t)row * a.lda + h] + a.dt_bias[h];
+        const float softplus = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+        cf[h] = expf(-expf(a.a_log[h]) * softplus);
+        cf[a.H + h] = 1.f / (1.f + expf(-a.beta[(size_t)row * a.ldb + h]));
     }
 }
 
@@ -146,10 +206,18 @@ extern "C" int cw_delta_prepare(const float* x, int ldx, const float* weight, in
     if (N < 0 || groups <= 0 || Dk <= 0 || H <= 0 || Dv <= 0 || taps <= 0 || ldx < 2 * groups * Dk + H * Dv || ldb < H || lda < H)
         return CW_ERR_BAD_SIZE;
     if (Dk > 32 * DP_CH) return CW_ERR_UNSUPPORTED;
+    const int C = 2 * groups * Dk + H * Dv;
+    auto whole = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const bool vec = taps == 4 && Dk % 4 == 0 && C % 4 == 0 && ldx % 4 == 0 && state_stride % 4 == 0 && conv_off % 4 == 0 && whole(x) &&
+                     whole(weight) && whole(state) && whole(out);
     int threads = 64;
-    while (threads < 256 && threads * 4 < 2 * groups * Dk + H * Dv) threads *= 2;
-    return cw_launch_ordered(delta_prepare_kernel, dim3(N), dim3(threads), 0, stream, x, ldx, weight, taps, state, state_stride, conv_off,
-                             slots, tok_seq, q_start, groups, Dk, H, Dv, eps, q_scale, beta, ldb, decay, lda, dt_bias, a_log, out, coef);
+    while (threads < 256 && threads * 4 < C) threads *= 2;
+    // few tokens: a token's channels over several blocks, as many as have work and fill the GPU once
+    int shares = 1;
+    while (shares < 32 && (long long)N * shares < 148 && shares * threads * 4 < C) shares *= 2;
+    const DeltaPrepareArgs args = {x, ldx, weight, taps, state, state_stride, conv_off, slots, tok_seq, q_start, groups, Dk, H, Dv, eps,
+                                   q_scale, beta, ldb, decay, lda, dt_bias, a_log, out, coef};
+    return cw_launch_ordered(vec ? delta_prepare_kernel<true> : delta_prepare_kernel<false>, dim3(N, shares), dim3(threads), 0, stream, args);
 }
 
 // ---- the delta rule ---------------------------------------------------------------------------------------
@@ -207,6 +275,8 @@ template <int IPT, bool HEAD>
 __global__ void __launch_bounds__(256)
 delta_scan_kernel(const DeltaScanArgs g) {
     extern __shared__ __align__(16) float ds_smem[];
+    __shared__ __align__(16) float nothing[4];  // zeros: what lanes without channels read
+    if (threadIdx.x < 4) nothing[threadIdx.x] = 0.f;
     pdl_wait();
     const int seq = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int start = g.q_start[seq], end = g.q_start[seq + 1];
@@ -229,6 +299,7 @@ delta_scan_kernel(const DeltaScanArgs g) {
     float* S_mem = row_state + g.state_off + ((size_t)h * Dv + (live ? j : 0)) * Dk;
     const int half = Dk >> 1;
     const bool mine = ipart * DS < Dk;  // (VEC: the thread owns channels at all)
+    const int token_step = mine ? Dk : 0, upper = mine ? half : 0;
     auto channel = [&](int r) { return VEC ? (r < 4 ? 0 : half) + ipart * 4 + (r & 3) : ipart + r * IP; };
     auto owns = [&](int r) { return VEC ? mine : ipart + r * IP < Dk; };
     float S[DS];
@@ -295,22 +366,20 @@ delta_scan_kernel(const DeltaScanArgs g) {
         __syncthreads();  // this chunk has landed; everyone has left the other buffer
         if (t0 + DC < end) fetch(t0 + DC, ds_smem + (which ^ 1) * buf_words);
         float part[DC];
-        auto token = [&](int t) {
+        const float* q0 = mine ? qs + ipart * 4 : nothing;
+        const float* k0 = mine ? ks + ipart * 4 : nothing;
+        const float* a0 = mine ? as + ipart * 4 : nothing;
+        auto token = [&](int t) {  // the thread's share of token t's output; its column of the state moves on by the token
             float kc[DS], qc[DS], ac[DS];
             if (VEC) {
-                const int at = t * Dk + ipart * 4, up = at + half;
-                if (mine) {
-                    *(float4*)&kc[0] = *(const float4*)(ks + at);
-                    *(float4*)&kc[4] = *(const float4*)(ks + up);
-                    *(float4*)&qc[0] = *(const float4*)(qs + at);
-                    *(float4*)&qc[4] = *(const float4*)(qs + up);
-                    if (!HEAD) {
-                        *(float4*)&ac[0] = *(const float4*)(as + at);
-                        *(float4*)&ac[4] = *(const float4*)(as + up);
-                    }
-                } else {
-#pragma unroll
-                    for (int r = 0; r < DS; ++r) kc[r] = qc[r] = ac[r] = 0.f;
+                const int at = t * token_step;
+                *(float4*)&kc[0] = *(const float4*)(k0 + at);
+                *(float4*)&kc[4] = *(const float4*)(k0 + at + upper);
+                *(float4*)&qc[0] = *(const float4*)(q0 + at);
+                *(float4*)&qc[4] = *(const float4*)(q0 + at + upper);
+                if (!HEAD) {
+                    *(float4*)&ac[0] = *(const float4*)(a0 + at);
+                    *(float4*)&ac[4] = *(const float4*)(a0 + at + upper);
                 }
             } else {
 #pragma unroll
@@ -357,29 +426,10 @@ delta_scan_kernel(const DeltaScanArgs g) {
             for (int t = 0; t < DC; ++t) part[t] = t < n ? token(t) : 0.f;
         }
         if (VEC) {
-            // tokens spread over the lanes while they are summed: a lane keeps one half of its tokens and hands the other on
-            int held = DC, first = 0;  // tokens this lane holds: first .. first + held - 1
+            const int first = sum_tokens_over_lanes<VEC ? IPT : 1, DC>(part, ipart);
+            if (live && first >= 0) {
 #pragma unroll
-            for (int o = IPT >> 1; o >= 1; o >>= 1) {
-                if (held > 1) {
-                    held >>= 1;
-                    const bool upper = (ipart & o) != 0;
-#pragma unroll
-                    for (int i = 0; i < DC / 2; ++i)
-                        if (i < held) {
-                            const float send = upper ? part[i] : part[i + held];
-                            const float keep = upper ? part[i + held] : part[i];
-                            part[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                        }
-                    if (upper) first += held;
-                } else {
-                    part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
-                }
-            }
-            constexpr int HELD = IPT > DC ? 1 : DC / (VEC ? IPT : 1);
-            if (live && (IPT <= DC || ipart % (IPT / DC > 0 ? IPT / DC : 1) == 0)) {
-#pragma unroll
-                for (int i = 0; i < HELD; ++i)
+                for (int i = 0; i < (IPT > DC ? 1 : DC / (VEC ? IPT : 1)); ++i)
                     if (first + i < n) g.out[(size_t)(t0 + first + i) * g.ldo + (size_t)h * Dv + j] = part[i];
             }
         } else {
