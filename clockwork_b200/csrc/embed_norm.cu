@@ -85,29 +85,6 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const T* __restric
 // The same for many rows (prompt portions): one warp per row, the row held in registers between the
 // sum of squares and the scaling, 16-byte accesses, no block-level synchronisation.  H must be a
 // multiple of 4 and at most 128 * NV.
-template <typename T>
-struct Vec4;
-template <>
-struct Vec4<float> {
-    static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
-    static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-};
-template <>
-struct Vec4<bf16> {
-    static __device__ __forceinline__ float4 load(const bf16* p) {
-        const uint2 r = *reinterpret_cast<const uint2*>(p);
-        const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&r.x), b = *reinterpret_cast<const __nv_bfloat162*>(&r.y);
-        return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
-    }
-    static __device__ __forceinline__ void store(bf16* p, float4 v) {
-        const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-        uint2 r;
-        r.x = *reinterpret_cast<const uint32_t*>(&a);
-        r.y = *reinterpret_cast<const uint32_t*>(&b);
-        *reinterpret_cast<uint2*>(p) = r;
-    }
-};
-
 // A row held in a warp's registers as v[i] = columns (i*32 + lane)*4 ..: takes the mean off every column that exists.
 template <int NV>
 __device__ __forceinline__ void warp_center(float4 (&v)[NV], int lane, int H) {

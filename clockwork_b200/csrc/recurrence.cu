@@ -529,21 +529,82 @@ gated_group_norm_kernel(const float* __restrict__ y, const float* __restrict__ z
     }
 }
 
+// The same with a warp per (row, part), four columns a lane and access, the part in registers between the two passes: parts of
+// a multiple of 4 columns, at most 128 * NV, at 16-byte addresses.
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+gated_group_norm_warp_kernel(const float* __restrict__ y, const float* __restrict__ z, int ldz, const float* __restrict__ weight,
+                             T* __restrict__ out, int N, int C, int parts, float eps, int mode) {
+    pdl_wait();
+    const bool ungated = mode & 8, gate_first = !ungated && (mode & 1), plain_sigmoid = mode & 2;
+    const int lane = threadIdx.x & 31;
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= (long long)N * parts) return;
+    const int row = (int)(item / parts), p = (int)(item - (long long)row * parts);
+    const int width = C / parts;
+    const float* yr = y + (size_t)row * C + (size_t)p * width;
+    const float* zr = z + (size_t)row * ldz + (size_t)p * width;
+    const float* wr = weight != nullptr ? weight + ((mode & 4) ? 0 : (size_t)p * width) : nullptr;
+    auto gate = [&](float g) { return (plain_sigmoid ? 1.f : g) / (1.f + expf(-g)); };
+    float4 u[NV], g[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = (i * 32 + lane) * 4;
+        if (c < width) {
+            u[i] = Vec4<float>::load(yr + c);
+            if (ungated) {
+                g[i] = make_float4(1.f, 1.f, 1.f, 1.f);
+            } else {
+                const float4 raw = Vec4<float>::load(zr + c);
+                g[i] = make_float4(gate(raw.x), gate(raw.y), gate(raw.z), gate(raw.w));
+            }
+            if (gate_first) u[i] = make_float4(u[i].x * g[i].x, u[i].y * g[i].y, u[i].z * g[i].z, u[i].w * g[i].w);
+            ss = fmaf(u[i].x, u[i].x, fmaf(u[i].y, u[i].y, fmaf(u[i].z, u[i].z, fmaf(u[i].w, u[i].w, ss))));
+        }
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)width + eps);
+    T* o = out + (size_t)row * C + (size_t)p * width;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = (i * 32 + lane) * 4;
+        if (c < width) {
+            float4 r = make_float4(u[i].x * inv, u[i].y * inv, u[i].z * inv, u[i].w * inv);
+            if (wr != nullptr) {
+                const float4 w = Vec4<float>::load(wr + c);
+                r = make_float4(r.x * w.x, r.y * w.y, r.z * w.z, r.w * w.w);
+            }
+            if (!gate_first) r = make_float4(r.x * g[i].x, r.y * g[i].y, r.z * g[i].z, r.w * g[i].w);
+            Vec4<T>::store(o + c, r);
+        }
+    }
+}
+
+template <typename T>
+static int launch_gated_group_norm(const float* y, const float* z, int ldz, const float* weight, T* out, int N, int C, int parts, float eps,
+                                   int mode, cudaStream_t stream) {
+    const int width = C / parts;
+    auto whole = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    if (width % 4 == 0 && width <= 1024 && C % 4 == 0 && ldz % 4 == 0 && whole(y) && whole(z) && whole(weight) && whole(out)) {
+        const dim3 grid((unsigned)(((long long)N * parts + 7) / 8));
+        const auto kernel = width <= 128   ? gated_group_norm_warp_kernel<T, 1>
+                            : width <= 256 ? gated_group_norm_warp_kernel<T, 2>
+                            : width <= 512 ? gated_group_norm_warp_kernel<T, 4>
+                                           : gated_group_norm_warp_kernel<T, 8>;
+        return cw_launch_ordered(kernel, grid, dim3(256), 0, stream, y, z, ldz, weight, out, N, C, parts, eps, mode);
+    }
+    int threads = 32;
+    while (threads < 256 && threads * 4 < width) threads *= 2;
+    return cw_launch_ordered(gated_group_norm_kernel<T>, dim3(N, parts), dim3(threads), 0, stream, y, z, ldz, weight, out, C, parts, eps, mode);
+}
+
 extern "C" int cw_gated_group_norm(const float* y, const float* z, int ldz, const float* weight, void* out, int N, int C,
                                    int parts, float eps, int mode, int dtype, cudaStream_t stream) {
     if (N == 0) return CW_OK;
     if (N < 0 || C <= 0 || parts <= 0 || C % parts || parts > 65535) return CW_ERR_BAD_SIZE;
     if (!(mode & 8) && (z == nullptr || ldz < C)) return CW_ERR_BAD_SIZE;
-    const int width = C / parts;
-    int threads = 32;
-    while (threads < 256 && threads * 4 < width) threads *= 2;
-    dim3 grid(N, parts);
-    if (dtype == 0)
-        return cw_launch_ordered(gated_group_norm_kernel<float>, grid, dim3(threads), 0, stream, y, z, ldz, weight, (float*)out, C, parts,
-                         eps, mode);
-    if (dtype == 1)
-        return cw_launch_ordered(gated_group_norm_kernel<bf16>, grid, dim3(threads), 0, stream, y, z, ldz, weight, (bf16*)out, C, parts,
-                         eps, mode);
+    if (dtype == 0) return launch_gated_group_norm<float>(y, z, ldz, weight, (float*)out, N, C, parts, eps, mode, stream);
+    if (dtype == 1) return launch_gated_group_norm<bf16>(y, z, ldz, weight, (bf16*)out, N, C, parts, eps, mode, stream);
     return CW_ERR_BAD_DTYPE;
 }
 

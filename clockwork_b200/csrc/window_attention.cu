@@ -72,8 +72,10 @@ extern "C" int cw_store_rows(const void* src, int ld, int col0, int width, void*
 // [H*dk] and k_norm [G*dk] the queries are first divided by the root mean square (eps inside the root) of all H*dk of them
 // and multiplied by q_norm, the keys likewise over their G*dk entries.  Then the leading entries of every query and key
 // head are rotated, everything in float32.  Queries go to q_out [N, H*dk], the rows [key | value] to the cache row that
-// the token's slot names (slots null or < 0: nothing is stored).
-template <typename T, bool NORM>
+// the token's slot names (slots null or < 0: nothing is stored).  Blocks: (token, share of its entries; each share forms
+// the norms' sums again).  VEC: four neighbouring entries at a time, 16-byte accesses (head sizes a multiple of 4 entries,
+// rotated ones of 4 or, with half pairs, of 8).
+template <typename T, bool NORM, bool VEC>
 __global__ void __launch_bounds__(256)
 rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict__ positions, const int* __restrict__ tok_seq,
                     const int* __restrict__ slots, Rotation rot, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
@@ -83,10 +85,11 @@ rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict
     __shared__ float scratch[33];
     pdl_wait();
     const int n = blockIdx.x;
+    const int at = blockIdx.y * blockDim.x + threadIdx.x, step = gridDim.y * blockDim.x;
     const int HQ = H * dk, row = dk + dv, half = rot.dims >> 1;
     T* qo = q_out + (size_t)n * HQ;
     if (tok_seq[n] < 0) {  // padding of a fixed-shape step
-        for (int c = threadIdx.x; c < HQ; c += blockDim.x) qo[c] = from_f<T>(0.f);
+        for (int c = at; c < HQ; c += step) qo[c] = from_f<T>(0.f);
         return;
     }
     const float* x = src + (size_t)n * ld;
@@ -97,12 +100,22 @@ rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict
     float q_inv = 1.f, k_inv = 1.f;
     if (NORM) {
         float qs = 0.f, ks = 0.f;
-        for (int c = threadIdx.x; c < HQ; c += blockDim.x) qs = fmaf(x[c], x[c], qs);
-        for (int g = 0; g < G; ++g)
-            for (int i = threadIdx.x; i < dk; i += blockDim.x) {
-                const float k = kv[(size_t)g * row + i];
-                ks = fmaf(k, k, ks);
+        if (VEC) {
+            auto square = [](float4 v, float s) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, s)))); };
+            for (int c = threadIdx.x * 4; c < HQ; c += blockDim.x * 4) qs = square(Vec4<float>::load(x + c), qs);
+            const int quads = dk >> 2;
+            for (int c = threadIdx.x; c < G * quads; c += blockDim.x) {
+                const int g = c / quads;
+                ks = square(Vec4<float>::load(kv + (size_t)g * row + (c - g * quads) * 4), ks);
             }
+        } else {
+            for (int c = threadIdx.x; c < HQ; c += blockDim.x) qs = fmaf(x[c], x[c], qs);
+            for (int g = 0; g < G; ++g)
+                for (int i = threadIdx.x; i < dk; i += blockDim.x) {
+                    const float k = kv[(size_t)g * row + i];
+                    ks = fmaf(k, k, ks);
+                }
+        }
         q_inv = 1.0f / sqrtf(block_sum(qs, scratch) / (float)HQ + eps);
         k_inv = 1.0f / sqrtf(block_sum(ks, scratch) / (float)(G * dk) + eps);
     }
@@ -125,18 +138,60 @@ rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict
         const float a = normed(i), b = normed(other);
         return first ? a * cs[pair] - b * sn[pair] : a * cs[pair] + b * sn[pair];
     };
-    for (int c = threadIdx.x; c < HQ; c += blockDim.x) {
-        const int h = c / dk, i = c - h * dk;
-        qo[c] = from_f<T>(entry(x + (size_t)h * dk, NORM ? q_norm + (size_t)h * dk : nullptr, q_inv, i));
+    // the same for entries i .. i + 3
+    auto entries = [&](const float* head, const float* w, float inv, int i) {
+        auto normed = [&](int e) {
+            float4 v = Vec4<float>::load(head + e);
+            if (NORM) {
+                const float4 g = Vec4<float>::load(w + e);
+                v = make_float4(v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z, v.w * inv * g.w);
+            }
+            return v;
+        };
+        const float4 a = normed(i);
+        if (i >= rot.dims) return a;
+        if (rot.interleaved) {
+            const int p = i >> 1;
+            return make_float4(a.x * cs[p] - a.y * sn[p], a.y * cs[p] + a.x * sn[p], a.z * cs[p + 1] - a.w * sn[p + 1],
+                               a.w * cs[p + 1] + a.z * sn[p + 1]);
+        }
+        const bool first = i < half;
+        const int p = first ? i : i - half;
+        const float4 b = normed(first ? i + half : i - half);
+        const float sign = first ? -1.f : 1.f;
+        return make_float4(a.x * cs[p] + b.x * (sign * sn[p]), a.y * cs[p + 1] + b.y * (sign * sn[p + 1]),
+                           a.z * cs[p + 2] + b.z * (sign * sn[p + 2]), a.w * cs[p + 3] + b.w * (sign * sn[p + 3]));
+    };
+    if (VEC) {
+        const int quads = dk >> 2;
+        for (int c = at; c < H * quads; c += step) {
+            const int h = c / quads, i = (c - h * quads) * 4;
+            Vec4<T>::store(qo + (size_t)h * dk + i, entries(x + (size_t)h * dk, NORM ? q_norm + (size_t)h * dk : nullptr, q_inv, i));
+        }
+    } else {
+        for (int c = at; c < HQ; c += step) {
+            const int h = c / dk, i = c - h * dk;
+            qo[c] = from_f<T>(entry(x + (size_t)h * dk, NORM ? q_norm + (size_t)h * dk : nullptr, q_inv, i));
+        }
     }
     const int slot = slots != nullptr ? slots[n] : -1;
     if (slot < 0) return;
     if (slot >= total_rows) {
-        if (threadIdx.x == 0) cw_report(status, CW_ST_SLOT_RANGE, n, slot);
+        if (at == 0) cw_report(status, CW_ST_SLOT_RANGE, n, slot);
         return;
     }
     T* to = cache + (size_t)slot * G * row;
-    for (int c = threadIdx.x; c < G * row; c += blockDim.x) {
+    if (VEC) {
+        const int quads = row >> 2;
+        for (int c = at; c < G * quads; c += step) {
+            const int g = c / quads, i = (c - g * quads) * 4;
+            const float* head = kv + (size_t)g * row;
+            Vec4<T>::store(to + (size_t)g * row + i, i < dk ? entries(head, NORM ? k_norm + (size_t)g * dk : nullptr, k_inv, i)
+                                                            : Vec4<float>::load(head + i));
+        }
+        return;
+    }
+    for (int c = at; c < G * row; c += step) {
         const int g = c / row, i = c - g * row;
         to[c] = from_f<T>(i < dk ? entry(kv + (size_t)g * row, NORM ? k_norm + (size_t)g * dk : nullptr, k_inv, i) : kv[c]);
     }
@@ -152,17 +207,26 @@ extern "C" int cw_rotate_store(const float* src, int ld, const int* positions, c
         (q_norm == nullptr) != (k_norm == nullptr))
         return CW_ERR_BAD_SIZE;
     if (rot_dims > 8192) return CW_ERR_UNSUPPORTED;
+    auto whole = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+    const bool vec = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 && rot_dims % (interleaved ? 4 : 8) == 0 && whole(src) && whole(q_out) &&
+                     whole(cache) && whole(q_norm) && whole(k_norm);
+    const int items = (H * dk + G * (dk + dv)) / (vec ? 4 : 1);
     int threads = 64;
-    while (threads < 256 && threads < H * dk) threads *= 2;
+    while (threads < 256 && threads < items) threads *= 2;
+    // few tokens: a token's entries over several blocks, as many as have work and fill the GPU once
+    int shares = 1;
+    while (shares < 16 && (long long)N * shares < 148 && shares * threads < items) shares *= 2;
     const size_t smem = sizeof(float) * (size_t)rot_dims;
-    const dim3 grid(N), block(threads);
+    const dim3 grid(N, shares), block(threads);
     if (dtype == 0) {
-        const auto kernel = q_norm != nullptr ? rotate_store_kernel<float, true> : rotate_store_kernel<float, false>;
+        const auto kernel = q_norm != nullptr ? (vec ? rotate_store_kernel<float, true, true> : rotate_store_kernel<float, true, false>)
+                                              : (vec ? rotate_store_kernel<float, false, true> : rotate_store_kernel<float, false, false>);
         return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv,
                                  (float*)q_out, (float*)cache, total_rows, status);
     }
     if (dtype == 1) {
-        const auto kernel = q_norm != nullptr ? rotate_store_kernel<bf16, true> : rotate_store_kernel<bf16, false>;
+        const auto kernel = q_norm != nullptr ? (vec ? rotate_store_kernel<bf16, true, true> : rotate_store_kernel<bf16, true, false>)
+                                              : (vec ? rotate_store_kernel<bf16, false, true> : rotate_store_kernel<bf16, false, false>);
         return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv,
                                  (bf16*)q_out, (bf16*)cache, total_rows, status);
     }
