@@ -216,11 +216,13 @@ recurrence_scan_kernel(const float* __restrict__ q, int ldq, const float* __rest
     pdl_wait();
     constexpr bool VEC = IPT > 0;
     const int IP = VEC ? IPT : ip;
-    const int seq = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    // (the request is the slowest index: the blocks of a request that brings tokens then start side by side on as many SMs,
+    // however many requests of a fixed-shape step bring none)
+    const int seq = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
     const int start = q_start[seq], end = q_start[seq + 1];
     if (end <= start) return;
     const int ipart = tid % IP, jl = tid / IP, JB = blockDim.x / IP;
-    const int j0 = blockIdx.z * JB, j = j0 + jl;
+    const int j0 = blockIdx.x * JB, j = j0 + jl;
     const bool live = j < Dv;
     if (tok_seq[start] < 0) {  // padding rows of a fixed-shape step: no request, no state
         if (live && ipart == 0)
@@ -400,7 +402,7 @@ extern "C" int cw_recurrence_scan(int form, const float* q, int ldq, const float
                                   float q_scale, cudaStream_t stream) {
     if (S == 0) return CW_OK;
     if (S < 0 || H <= 0 || Dk <= 0 || Dv <= 0 || heads_per_group <= 0 || H % heads_per_group) return CW_ERR_BAD_SIZE;
-    if (Dk > 32 * RS || H > 65535) return CW_ERR_UNSUPPORTED;
+    if (Dk > 32 * RS || H > 65535 || S > 65535) return CW_ERR_UNSUPPORTED;
     int IP = 1, log_ip = 0;
     while (IP * RS < Dk) {
         IP *= 2;
@@ -409,7 +411,7 @@ extern "C" int cw_recurrence_scan(int form, const float* q, int ldq, const float
     int threads = 256;  // more value columns per block share the staged q and k; fewer when a head has few columns
     while (threads > 32 && threads / IP >= 2 * Dv) threads /= 2;
     const int JB = threads / IP;
-    dim3 grid(S, H, (Dv + JB - 1) / JB);
+    dim3 grid((Dv + JB - 1) / JB, H, S);
     if (form < 0 || form > 4) return CW_ERR_UNSUPPORTED;
     if (form == 4 && Dv < 2) return CW_ERR_BAD_SIZE;
     const bool ch = form == 0 || form == 2;  // coefficients per key channel

@@ -278,13 +278,15 @@ delta_scan_kernel(const DeltaScanArgs g) {
     __shared__ __align__(16) float nothing[4];  // zeros: what lanes without channels read
     if (threadIdx.x < 4) nothing[threadIdx.x] = 0.f;
     pdl_wait();
-    const int seq = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+    // (the request is the slowest index: the blocks of a request that brings tokens then start side by side on as many SMs,
+    // however many requests of a fixed-shape step bring none)
+    const int seq = blockIdx.z, h = blockIdx.y, tid = threadIdx.x;
     const int start = g.q_start[seq], end = g.q_start[seq + 1];
     if (end <= start) return;
     constexpr bool VEC = IPT > 0;
     const int IP = VEC ? IPT : g.IP, Dk = g.Dk, Dv = g.Dv;
     const int ipart = tid % IP, jl = tid / IP, JB = blockDim.x / IP;
-    const int j0 = blockIdx.z * JB, j = j0 + jl;
+    const int j0 = blockIdx.x * JB, j = j0 + jl;
     const bool live = j < Dv;
     if (g.tok_seq[start] < 0) {  // padding rows of a fixed-shape step: no request, no state
         if (live && ipart == 0)
@@ -346,7 +348,7 @@ delta_scan_kernel(const DeltaScanArgs g) {
     };
     fetch(start, ds_smem);
     if (g.carry != nullptr) {  // the blocks of the request share its channels out
-        const int n = end - start, block = blockIdx.y * gridDim.z + blockIdx.z, blocks = gridDim.y * gridDim.z;
+        const int n = end - start, block = blockIdx.y * gridDim.x + blockIdx.x, blocks = gridDim.y * gridDim.x;
         float* kept = row_state + g.carry_off;
         for (int c = block * blockDim.x + tid; c < g.C; c += blocks * blockDim.x)
             for (int d = g.R; d >= 1; --d)  // ascending writes; what is read lies ahead of what was written
@@ -460,7 +462,7 @@ extern "C" int cw_delta_scan(const float* q, int ldq, const float* k, int ldk, c
     if (S == 0) return CW_OK;
     if (S < 0 || H <= 0 || Dk <= 0 || Dv <= 0 || heads_per_group <= 0 || H % heads_per_group) return CW_ERR_BAD_SIZE;
     if (carry != nullptr && (C <= 0 || R < 0 || ldc < C)) return CW_ERR_BAD_SIZE;
-    if (Dk > 32 * DS || H > 65535) return CW_ERR_UNSUPPORTED;
+    if (Dk > 32 * DS || H > 65535 || S > 65535) return CW_ERR_UNSUPPORTED;
     int IP = 1, log_ip = 0;
     while (IP * DS < Dk) {
         IP *= 2;
@@ -469,7 +471,7 @@ extern "C" int cw_delta_scan(const float* q, int ldq, const float* k, int ldk, c
     int threads = 256;  // more value columns per block share the staged q, k and decays; fewer when a head has few columns
     while (threads > 32 && threads / IP >= 2 * Dv) threads /= 2;
     const int JB = threads / IP;
-    dim3 grid(S, H, (Dv + JB - 1) / JB);
+    dim3 grid((Dv + JB - 1) / JB, H, S);
     const int wide = Dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k & 15) == 0 &&
                      (head_decay || (lda % 4 == 0 && ((uintptr_t)a & 15) == 0));
     const bool vec = wide && Dk % DS == 0;
