@@ -120,6 +120,14 @@ __device__ __forceinline__ int sum_tokens_over_lanes(float (&part)[TOKENS], int 
     return first;
 }
 
+// Dynamic shared memory that a scan over a long portion asks for so that no two of its blocks share an SM: a step of `rows`
+// rows whose grid holds blocks for requests that bring none must not put two of the blocks that do work side by side while
+// other SMs idle.  Short steps keep what they need.
+static inline size_t cw_scan_smem(size_t needed, long long rows) {
+    const size_t alone = 120u << 10;
+    return rows >= 256 && needed < alone ? alone : needed;
+}
+
 // Block-wide reductions with a fixed order (warp tree, then warp 0 over the warp results),
 // so the result for a row never depends on what else is in the batch.
 // `scratch` must hold 33 floats.  All threads receive the result.

@@ -394,12 +394,13 @@ recurrence_scan_kernel(const float* __restrict__ q, int ldq, const float* __rest
     }
 }
 
+// rows: the rows of the step (all requests'), which only sizes the blocks.
 // pre: the coefficients that cw_recurrence_coefficients made (form 0: a [N, H*Dk]; form 1: [a | dt] [N, 2H]).
 extern "C" int cw_recurrence_scan(int form, const float* q, int ldq, const float* k, int ldk, const float* v, int ldv,
                                   const float* pre, int ldp, const float* p0, const float* p1, const float* p2,
                                   float* state, long long state_stride, long long state_off, const long long* slots,
                                   const int* tok_seq, const int* q_start, int S, int H, int Dk, int Dv, int heads_per_group, float* out, int ldo,
-                                  float q_scale, cudaStream_t stream) {
+                                  float q_scale, int rows, cudaStream_t stream) {
     if (S == 0) return CW_OK;
     if (S < 0 || H <= 0 || Dk <= 0 || Dv <= 0 || heads_per_group <= 0 || H % heads_per_group) return CW_ERR_BAD_SIZE;
     if (Dk > 32 * RS || H > 65535 || S > 65535) return CW_ERR_UNSUPPORTED;
@@ -418,7 +419,7 @@ extern "C" int cw_recurrence_scan(int form, const float* q, int ldq, const float
     if ((form != 3 && pre == nullptr) || (form == 3 && p0 == nullptr)) return CW_ERR_BAD_SIZE;
     const int wide = Dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && (!ch || ldp % 4 == 0) && ((uintptr_t)q & 15) == 0 &&
                      ((uintptr_t)k & 15) == 0 && (!ch || ((uintptr_t)pre & 15) == 0);
-    const size_t smem = 2 * sizeof(float) * (size_t)(2 * RC * Dk + (ch ? RC * Dk : (form == 1 || form == 4 ? 2 * RC : 0)) + RC * JB);
+    const size_t smem = cw_scan_smem(2 * sizeof(float) * (size_t)(2 * RC * Dk + (ch ? RC * Dk : (form == 1 || form == 4 ? 2 * RC : 0)) + RC * JB), rows);
     const int which = wide && Dk % RS == 0 ? log_ip : 6;
     static size_t allowed[5][7] = {};
     using Kernel = void (*)(const float*, int, const float*, int, const float*, int, const float*, int, const float*, const float*,

@@ -453,12 +453,12 @@ delta_scan_kernel(const DeltaScanArgs g) {
 }
 
 // q, k [N, groups*Dk] (head h reads group h / heads_per_group), v [N, H*Dv], beta [N, H], decays a [N, H*Dk] or, with
-// head_decay, [N, H]: float32, unit column stride, any row stride.  out [N, H*Dv].
+// head_decay, [N, H]: float32, unit column stride, any row stride.  out [N, H*Dv].  rows: N, which only sizes the blocks.
 extern "C" int cw_delta_scan(const float* q, int ldq, const float* k, int ldk, const float* v, int ldv, const float* a, int lda,
                              int head_decay, const float* beta, int ldb, float* state, long long state_stride, long long state_off,
                              const long long* slots, const int* tok_seq, const int* q_start, int S, int H, int Dk, int Dv,
                              int heads_per_group, float* out, int ldo, const float* carry, int ldc, int C, int R, long long carry_off,
-                             cudaStream_t stream) {
+                             int rows, cudaStream_t stream) {
     if (S == 0) return CW_OK;
     if (S < 0 || H <= 0 || Dk <= 0 || Dv <= 0 || heads_per_group <= 0 || H % heads_per_group) return CW_ERR_BAD_SIZE;
     if (carry != nullptr && (C <= 0 || R < 0 || ldc < C)) return CW_ERR_BAD_SIZE;
@@ -475,7 +475,7 @@ extern "C" int cw_delta_scan(const float* q, int ldq, const float* k, int ldk, c
     const int wide = Dk % 4 == 0 && ldq % 4 == 0 && ldk % 4 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k & 15) == 0 &&
                      (head_decay || (lda % 4 == 0 && ((uintptr_t)a & 15) == 0));
     const bool vec = wide && Dk % DS == 0;
-    const size_t smem = 2 * sizeof(float) * (size_t)((head_decay ? 2 : 3) * DC * Dk + DC * JB + (head_decay ? 2 : 1) * DC);
+    const size_t smem = cw_scan_smem(2 * sizeof(float) * (size_t)((head_decay ? 2 : 3) * DC * Dk + DC * JB + (head_decay ? 2 : 1) * DC), rows);
     using Kernel = void (*)(const DeltaScanArgs);
     static const Kernel kernels[2][7] = {
         {delta_scan_kernel<1, false>, delta_scan_kernel<2, false>, delta_scan_kernel<4, false>, delta_scan_kernel<8, false>,

@@ -34,7 +34,7 @@ _SIGNATURES: dict[str, list] = {
     "cw_shift_mix": [P, P, P, LL, LL, P, P, P, P, I, I, I, I, P],
     "cw_causal_conv": [P, I, P, P, P, LL, LL, P, P, P, P, I, I, I, P],
     "cw_carry_rows": [P, I, P, LL, LL, P, P, P, I, I, I, I, P],
-    "cw_recurrence_scan": [I, P, I, P, I, P, I, P, I, P, P, P, P, LL, LL, P, P, P, I, I, I, I, I, P, I, F, P],
+    "cw_recurrence_scan": [I, P, I, P, I, P, I, P, I, P, P, P, P, LL, LL, P, P, P, I, I, I, I, I, P, I, F, I, P],
     "cw_sigmoid_power_decay": [P, I, I, I, F, P],
     "cw_activation_cols": [P, I, I, I, I, I, P],
     "cw_recurrence_coefficients": [I, P, I, P, P, P, I, I, P],
@@ -68,7 +68,7 @@ _SIGNATURES: dict[str, list] = {
     "cw_unit_heads": [P, I, I, I, I, F, I, F, F, P],
     "cw_delta_coefficients": [P, I, P, P, P, I, I, I, I, P],
     "cw_delta_prepare": [P, I, P, I, P, LL, LL, P, P, P, I, I, I, I, F, F, P, I, P, I, P, P, I, P, P, P],
-    "cw_delta_scan": [P, I, P, I, P, I, P, I, I, P, I, P, LL, LL, P, P, P, I, I, I, I, I, P, I, P, I, I, I, LL, P],
+    "cw_delta_scan": [P, I, P, I, P, I, P, I, I, P, I, P, LL, LL, P, P, P, I, I, I, I, I, P, I, P, I, I, I, LL, I, P],
     "cw_gate_scan": [P, I, P, I, P, P, F, P, LL, LL, P, P, P, I, I, I, P, P],
     "cw_memory_norm": [P, P, I, P, I, P, P, I, I, I, F, I, P],
     # attention over a cached latent (csrc/latent_attention.cu)

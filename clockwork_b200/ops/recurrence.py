@@ -95,7 +95,7 @@ def recurrence_scan(form: int, q, k, v, pre, p0, p1, p2, view, offset: int, ctx,
         pre = coef
     check(library().cw_recurrence_scan(form, _ptr(q), ld(q), _ptr(k), ld(k), _ptr(v), ld(v), _ptr(pre), 0 if pre is None else ld(pre),
                                        _ptr(p0), _ptr(p1), _ptr(p2), state, stride, offset, slots, _ptr(ctx.tok_seq), _ptr(ctx.q_start),
-                                       ctx.num_seqs, heads, dk, dv, heads_per_group, _ptr(out), heads * dv, float(q_scale), _stream()),
+                                       ctx.num_seqs, heads, dk, dv, heads_per_group, _ptr(out), heads * dv, float(q_scale), n, _stream()),
           "recurrence_scan")
     return out
 
@@ -135,7 +135,7 @@ def delta_scan(q, k, v, pre, beta, dt_bias, a_log, view, offset: int, ctx, heads
           "delta_coefficients")
     check(library().cw_delta_scan(_ptr(q), ld(q), _ptr(k), ld(k), _ptr(v), ld(v), _ptr(pre), ld(pre), 0, _ptr(beta), ld(beta), state, stride,
                                   offset, slots, _ptr(ctx.tok_seq), _ptr(ctx.q_start), ctx.num_seqs, heads, dk, dv, heads_per_group,
-                                  _ptr(out), heads * dv, None, 0, 0, 0, 0, _stream()), "delta_scan")
+                                  _ptr(out), heads * dv, None, 0, 0, 0, 0, n, _stream()), "delta_scan")
     return out
 
 
@@ -175,7 +175,7 @@ def head_delta(x, conv_weight, beta, decay, dt_bias, a_log, view, scan_offset: i
     check(library().cw_delta_scan(_ptr(qkv), channels, _ptr(qkv[:, qk:]), channels, _ptr(qkv[:, 2 * qk :]), channels, _ptr(coef), 2 * heads, 1,
                                   _ptr(coef[:, heads:]), 2 * heads, state, stride, scan_offset, slots, _ptr(ctx.tok_seq), _ptr(ctx.q_start),
                                   ctx.num_seqs, heads, dk, dv, heads // groups, _ptr(out), heads * dv, _ptr(x), ld(x), channels, taps - 1,
-                                  conv_offset, _stream()), "delta_scan")
+                                  conv_offset, n, _stream()), "delta_scan")
     return out
 
 
