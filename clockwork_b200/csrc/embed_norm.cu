@@ -38,11 +38,12 @@ extern "C" int cw_embed(float* out, const void* table, const int* ids, int N, in
 
 // resid[row] (+= delta[row]); out[r] = weight * (x * rsqrt(mean(x^2)+eps)).
 // With `rows` given, output row r is computed from residual row rows[r] (no add is done).  CENTER: x - mean(x) in x's place.
+// `out2` (or null): the same normalised row times a second weight.
 template <typename T, bool CENTER>
 __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const T* __restrict__ delta,
                                    const float* __restrict__ weight, T* __restrict__ out,
                                    const int* __restrict__ rows, int num_resid_rows, float eps,
-                                   int H, int* status) {
+                                   int H, int* status, const float* __restrict__ weight2, T* __restrict__ out2) {
     __shared__ float scratch[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -79,7 +80,11 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ resid, const T* __restric
     ss = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(ss / (float)H + eps);
     T* o = out + (size_t)r * H;
-    for (int c = threadIdx.x; c < H; c += blockDim.x) o[c] = from_f<T>(weight[c] * ((CENTER ? x[c] - mean : x[c]) * inv));
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        const float v = (CENTER ? x[c] - mean : x[c]) * inv;
+        o[c] = from_f<T>(weight[c] * v);
+        if (out2 != nullptr) out2[(size_t)r * H + c] = from_f<T>(weight2[c] * v);
+    }
 }
 
 // The same for many rows (prompt portions): one warp per row, the row held in registers between the
@@ -114,7 +119,7 @@ __device__ __forceinline__ float warp_square_sum(const float4 (&v)[NV], int lane
 template <typename T, int NV, bool CENTER>
 __global__ void __launch_bounds__(256)
 add_rmsnorm_warp_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ weight,
-                        T* __restrict__ out, int num_rows, float eps, int H) {
+                        T* __restrict__ out, int num_rows, float eps, int H, const float* __restrict__ weight2, T* __restrict__ out2) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -145,18 +150,22 @@ add_rmsnorm_warp_kernel(float* __restrict__ resid, const T* __restrict__ delta, 
         if (c < H) {
             const float4 w = Vec4<float>::load(weight + c);
             Vec4<T>::store(o + c, make_float4(w.x * (v[i].x * inv), w.y * (v[i].y * inv), w.z * (v[i].z * inv), w.w * (v[i].w * inv)));
+            if (out2 != nullptr) {
+                const float4 u = Vec4<float>::load(weight2 + c);
+                Vec4<T>::store(out2 + (size_t)r * H + c, make_float4(u.x * (v[i].x * inv), u.y * (v[i].y * inv), u.z * (v[i].z * inv), u.w * (v[i].w * inv)));
+            }
         }
     }
 }
 
 template <typename T, bool CENTER>
 static int launch_rmsnorm_warp(float* resid, const T* delta, const float* weight, T* out, int rows, int H, float eps,
-                               cudaStream_t stream) {
+                               const float* weight2, T* out2, cudaStream_t stream) {
     const int warps = 8;
     const dim3 grid((rows + warps - 1) / warps), block(warps * 32);
     const int nv = (H + 127) / 128;
 #define CW_NV(n) \
-    if (nv <= n) return cw_launch(add_rmsnorm_warp_kernel<T, n, CENTER>, grid, block, 0, stream, 1, resid, delta, weight, out, rows, eps, H);
+    if (nv <= n) return cw_launch(add_rmsnorm_warp_kernel<T, n, CENTER>, grid, block, 0, stream, 1, resid, delta, weight, out, rows, eps, H, weight2, out2);
     CW_NV(4) CW_NV(8) CW_NV(12) CW_NV(16) CW_NV(24) CW_NV(32)
 #undef CW_NV
     return CW_ERR_UNSUPPORTED;
@@ -164,34 +173,35 @@ static int launch_rmsnorm_warp(float* resid, const T* delta, const float* weight
 
 template <typename T, bool CENTER>
 static int launch_add_rmsnorm(float* resid, const T* delta, const float* weight, T* out, const int* rows, int num_out_rows,
-                              int num_resid_rows, int H, float eps, int* status, cudaStream_t stream) {
+                              int num_resid_rows, int H, float eps, int* status, const float* weight2, T* out2, cudaStream_t stream) {
     // many rows: a warp per row; few rows (decode): a block per row, for the latency of the one row
     const bool aligned = H % 4 == 0 && H <= 4096 && ((uintptr_t)resid & 15) == 0 && ((uintptr_t)weight & 15) == 0 &&
-                         ((uintptr_t)out & 15) == 0 && ((uintptr_t)delta & 15) == 0;
+                         ((uintptr_t)out & 15) == 0 && ((uintptr_t)delta & 15) == 0 && ((uintptr_t)weight2 & 15) == 0 &&
+                         ((uintptr_t)out2 & 15) == 0;
     if (rows == nullptr && num_out_rows >= 256 && aligned)
-        return launch_rmsnorm_warp<T, CENTER>(resid, delta, weight, out, num_out_rows, H, eps, stream);
+        return launch_rmsnorm_warp<T, CENTER>(resid, delta, weight, out, num_out_rows, H, eps, weight2, out2, stream);
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     return cw_launch(add_rmsnorm_kernel<T, CENTER>, dim3(num_out_rows), dim3(threads), 0, stream, 1, resid, delta, weight, out, rows,
-                     num_resid_rows, eps, H, status);
+                     num_resid_rows, eps, H, status, weight2, out2);
 }
 
 // center: 0 RMSNorm, 1 layer norm
 extern "C" int cw_add_rmsnorm(float* resid, const void* delta, const float* weight, void* out,
                               const int* rows, int num_out_rows, int num_resid_rows, int H,
-                              float eps, int center, int dtype, int* status, cudaStream_t stream) {
+                              float eps, int center, int dtype, const float* weight2, void* out2, int* status, cudaStream_t stream) {
     if (num_out_rows == 0) return CW_OK;
-    if (num_out_rows < 0 || H <= 0) return CW_ERR_BAD_SIZE;
+    if (num_out_rows < 0 || H <= 0 || (out2 == nullptr) != (weight2 == nullptr)) return CW_ERR_BAD_SIZE;
     if (rows != nullptr && delta != nullptr) return CW_ERR_UNSUPPORTED;
     if (dtype == 0)
         return center ? launch_add_rmsnorm<float, true>(resid, (const float*)delta, weight, (float*)out, rows, num_out_rows, num_resid_rows, H,
-                                                        eps, status, stream)
+                                                        eps, status, weight2, (float*)out2, stream)
                       : launch_add_rmsnorm<float, false>(resid, (const float*)delta, weight, (float*)out, rows, num_out_rows, num_resid_rows, H,
-                                                         eps, status, stream);
+                                                         eps, status, weight2, (float*)out2, stream);
     if (dtype == 1)
         return center ? launch_add_rmsnorm<bf16, true>(resid, (const bf16*)delta, weight, (bf16*)out, rows, num_out_rows, num_resid_rows, H,
-                                                       eps, status, stream)
+                                                       eps, status, weight2, (bf16*)out2, stream)
                       : launch_add_rmsnorm<bf16, false>(resid, (const bf16*)delta, weight, (bf16*)out, rows, num_out_rows, num_resid_rows, H,
-                                                        eps, status, stream);
+                                                        eps, status, weight2, (bf16*)out2, stream);
     return CW_ERR_BAD_DTYPE;
 }
 
@@ -201,7 +211,8 @@ extern "C" int cw_add_rmsnorm(float* resid, const void* delta, const float* weig
 template <typename T, int NV, bool CENTER>
 __global__ void __launch_bounds__(256)
 add_parts_rmsnorm_kernel(float* __restrict__ resid, const float* __restrict__ parts, int num_parts, size_t part_stride,
-                         const float* __restrict__ weight, T* __restrict__ out, int num_rows, float eps, int H) {
+                         const float* __restrict__ weight, T* __restrict__ out, int num_rows, float eps, int H,
+                         const float* __restrict__ weight2, T* __restrict__ out2) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -241,18 +252,22 @@ add_parts_rmsnorm_kernel(float* __restrict__ resid, const float* __restrict__ pa
         if (c < H) {
             const float4 w = Vec4<float>::load(weight + c);
             Vec4<T>::store(o + c, make_float4(w.x * (v[i].x * inv), w.y * (v[i].y * inv), w.z * (v[i].z * inv), w.w * (v[i].w * inv)));
+            if (out2 != nullptr) {
+                const float4 u = Vec4<float>::load(weight2 + c);
+                Vec4<T>::store(out2 + (size_t)r * H + c, make_float4(u.x * (v[i].x * inv), u.y * (v[i].y * inv), u.z * (v[i].z * inv), u.w * (v[i].w * inv)));
+            }
         }
     }
 }
 
 template <typename T, bool CENTER>
 static int launch_add_parts(float* resid, const float* parts, int num_parts, size_t part_stride, const float* weight, T* out,
-                            int rows, int H, float eps, cudaStream_t stream) {
+                            int rows, int H, float eps, const float* weight2, T* out2, cudaStream_t stream) {
     const int warps = 8;
     const dim3 grid((rows + warps - 1) / warps), block(warps * 32);
     const int nv = (H + 127) / 128;
 #define CW_NV(n) \
-    if (nv <= n) return cw_launch(add_parts_rmsnorm_kernel<T, n, CENTER>, grid, block, 0, stream, 1, resid, parts, num_parts, part_stride, weight, out, rows, eps, H);
+    if (nv <= n) return cw_launch(add_parts_rmsnorm_kernel<T, n, CENTER>, grid, block, 0, stream, 1, resid, parts, num_parts, part_stride, weight, out, rows, eps, H, weight2, out2);
     CW_NV(4) CW_NV(8) CW_NV(12) CW_NV(16) CW_NV(24) CW_NV(32)
 #undef CW_NV
     return CW_ERR_UNSUPPORTED;
@@ -261,19 +276,22 @@ static int launch_add_parts(float* resid, const float* parts, int num_parts, siz
 // parts: float32 [num_parts][part_rows][H] (part_rows >= rows); out null: only the sum.  H a multiple of 4,
 // at most 4096; 16-byte aligned pointers; CW_ERR_UNSUPPORTED otherwise.
 extern "C" int cw_add_parts_rmsnorm(float* resid, const float* parts, int num_parts, int part_rows, const float* weight,
-                                    void* out, int rows, int H, float eps, int center, int dtype, cudaStream_t stream) {
+                                    void* out, int rows, int H, float eps, int center, int dtype, const float* weight2, void* out2,
+                                    cudaStream_t stream) {
     if (rows == 0) return CW_OK;
-    if (rows < 0 || H <= 0 || num_parts < 1 || part_rows < rows) return CW_ERR_BAD_SIZE;
+    if (rows < 0 || H <= 0 || num_parts < 1 || part_rows < rows || (out2 == nullptr) != (weight2 == nullptr) ||
+        (out2 != nullptr && out == nullptr))
+        return CW_ERR_BAD_SIZE;
     if (H % 4 != 0 || H > 4096 || ((uintptr_t)resid & 15) || ((uintptr_t)parts & 15) || ((uintptr_t)weight & 15) ||
-        ((uintptr_t)out & 15))
+        ((uintptr_t)out & 15) || ((uintptr_t)weight2 & 15) || ((uintptr_t)out2 & 15))
         return CW_ERR_UNSUPPORTED;
     const size_t stride = (size_t)part_rows * H;
     if (out == nullptr || (dtype == 0 && !center))
-        return launch_add_parts<float, false>(resid, parts, num_parts, stride, weight, (float*)out, rows, H, eps, stream);
-    if (dtype == 0) return launch_add_parts<float, true>(resid, parts, num_parts, stride, weight, (float*)out, rows, H, eps, stream);
+        return launch_add_parts<float, false>(resid, parts, num_parts, stride, weight, (float*)out, rows, H, eps, weight2, (float*)out2, stream);
+    if (dtype == 0) return launch_add_parts<float, true>(resid, parts, num_parts, stride, weight, (float*)out, rows, H, eps, weight2, (float*)out2, stream);
     if (dtype == 1)
-        return center ? launch_add_parts<bf16, true>(resid, parts, num_parts, stride, weight, (bf16*)out, rows, H, eps, stream)
-                      : launch_add_parts<bf16, false>(resid, parts, num_parts, stride, weight, (bf16*)out, rows, H, eps, stream);
+        return center ? launch_add_parts<bf16, true>(resid, parts, num_parts, stride, weight, (bf16*)out, rows, H, eps, weight2, (bf16*)out2, stream)
+                      : launch_add_parts<bf16, false>(resid, parts, num_parts, stride, weight, (bf16*)out, rows, H, eps, weight2, (bf16*)out2, stream);
     return CW_ERR_BAD_DTYPE;
 }
 

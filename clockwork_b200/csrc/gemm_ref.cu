@@ -10,7 +10,7 @@
 // within a few units in the last place of the exact dot product at any K.
 //
 // Epilogues: 0 store as T; 1 add into a float32 matrix (the residual stream); 2 store float32
-// (logits).  The SwiGLU variant computes silu(A Wg^T) * (A Wu^T) (clockwork/engine/model.py:62-63).
+// (logits); 4 store max(v, 0)^2 as T.  The SwiGLU variant computes silu(A Wg^T) * (A Wu^T) (clockwork/engine/model.py:62-63).
 #include "common.cuh"
 
 #define BM 64
@@ -104,6 +104,9 @@ gemm_ref_kernel(const T* __restrict__ A, const T* __restrict__ W, const T* __res
                 ((T*)Cout)[idx] = from_f<T>(g / (1.0f + expf(-g)) * u);
             } else if (epilogue == 0) {
                 ((T*)Cout)[idx] = from_f<T>(v);
+            } else if (epilogue == 4) {  // the square of what is positive
+                v = fmaxf(v, 0.f);
+                ((T*)Cout)[idx] = from_f<T>(v * v);
             } else if (epilogue == 1) {
                 ((float*)Cout)[idx] += v;
             } else {
@@ -118,7 +121,7 @@ extern "C" int cw_gemm_ref(const void* A, const void* W, const float* bias, void
                            cudaStream_t stream) {
     if (M == 0 || N == 0) return CW_OK;
     if (M < 0 || N < 0 || K <= 0 || lda < K || ldc < N) return CW_ERR_BAD_SIZE;
-    if (epilogue < 0 || epilogue > 2) return CW_ERR_UNSUPPORTED;
+    if (epilogue < 0 || (epilogue > 2 && epilogue != 4)) return CW_ERR_UNSUPPORTED;
     dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
     if (grid.y > 65535) return CW_ERR_BAD_SIZE;
     if (dtype == 0)

@@ -44,6 +44,7 @@ struct GemmParams {
     int T, N, K;          // tokens, output features, inner size
     int ldc;              // row stride of C in elements
     int epilogue;         // 0 bf16 store, 1 float32 add, 2 float32 store (ignored for SWIGLU);
+                          // (a call's epilogue 4 is 0 with squared_relu)
                           // 3 (CTA-pair kernel): float32 store of split ks at rows ks * part_rows .. of C
     int part_rows;        // epilogue 3: rows per split in C (the token count rounded up to the store's 16 rows)
     int num_kb;           // ceil(K / 64)
@@ -68,7 +69,13 @@ struct GemmParams {
     float* emit_part;         // [T, gridDim.x]
     int* split_flags;         // CTA-pair kernel with splits > 1: two words per tile, zero between launches
     float act_limit;          // SWIGLU only.  0: silu(gate) * up.  Positive: the clamped form (gated_act)
+    int squared_relu;         // not SWIGLU, epilogue 0: max(v, 0)^2 of v = product + bias is stored instead of v
 };
+
+__device__ __forceinline__ float squared_relu(float v) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+}
 
 // What the gated kernels make of the two accumulators.  limit 0: silu(g) * u.  limit > 0: with a = min(g, limit) and
 // b = clamp(u, -limit, limit), a * sigmoid(1.702 a) * (b + 1).  One straight line for both: without a limit the bounds
@@ -325,6 +332,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                 const float sc = scaled ? inv_s[c + j] : 1.0f;
                 float v = g[j] * sc + bias;
                 if (SWIGLU) v = gated_act(v, u[j] * sc, p.act_limit);
+                else if (p.squared_relu) v = squared_relu(v);
                 if (wide)
                     stage[(c + j) * BM + row] = v;
                 else
@@ -385,6 +393,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant_
                         if (j < ncols && t_base + j < p.T)
                             c16[(size_t)j * p.ldc] = __float2bfloat16_rn(gated_act(g[j], u[j], p.act_limit));
                 } else if (p.epilogue == 0) {
+                    if (p.squared_relu) {
+#pragma unroll
+                        for (int j = 0; j < NC; ++j) g[j] = squared_relu(g[j]);
+                    }
 #pragma unroll
                     for (int j = 0; j < NC; ++j)
                         if (j < ncols && t_base + j < p.T) c16[(size_t)j * p.ldc] = __float2bfloat16_rn(g[j]);
@@ -655,6 +667,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_w, const __gri
                 for (int j = 0; j < 16; ++j) {
                     float v = g[j] + bias;
                     if (SWIGLU) v = gated_act(v, u[j], p.act_limit);
+                    else if (p.squared_relu) v = squared_relu(v);
                     if (wide)
                         st32[j * BM + row] = v;
                     else
@@ -954,7 +967,8 @@ extern "C" int cw_gemm_tc_plan(int T, int N, int K, int swiglu, int sm_count, in
     return CW_OK;
 }
 
-// X [T, K] (row stride ldx), W [N, K] (and W2 for SwiGLU), C [T, ldc].  K must be a multiple of 8
+// X [T, K] (row stride ldx), W [N, K] (and W2 for SwiGLU), C [T, ldc].  Epilogues: 0 bfloat16 store, 1 add into float32, 2
+// float32 store, 4 bfloat16 store of max(v, 0)^2 (v: the product plus the bias).  K must be a multiple of 8
 // and all bases 16-byte aligned (TMA); returns CW_ERR_UNSUPPORTED otherwise so the caller can
 // use the plain kernel.
 //
@@ -997,11 +1011,13 @@ static int gemm_tc_run(const void* X, const void* W, const void* W2, const float
                        cudaStream_t stream) {
     if (T == 0 || N == 0) return CW_OK;
     if (T < 0 || N < 0 || K <= 0 || ldx < K || ldc < N) return CW_ERR_BAD_SIZE;
+    const bool swiglu = W2 != nullptr;
+    const bool relu2 = epilogue == 4 && !swiglu;
+    if (relu2) epilogue = 0;
     if (epilogue < 0 || epilogue > 2) return CW_ERR_UNSUPPORTED;
     if (K % 8 != 0 || ldx % 8 != 0 || ((uintptr_t)X & 15) || ((uintptr_t)W & 15) || ((uintptr_t)W2 & 15))
         return CW_ERR_UNSUPPORTED;
     if (load_encode() != 0) return CW_ERR_UNSUPPORTED;
-    const bool swiglu = W2 != nullptr;
     // C leaves through TMA when its rows are 16-byte multiples at a 16-byte base and the tile is not split
     const bool c_f32 = !swiglu && epilogue != 0;
     const long long c_row_bytes = (long long)ldc * (c_f32 ? 4 : 2);
@@ -1032,6 +1048,7 @@ static int gemm_tc_run(const void* X, const void* W, const void* W2, const float
     p.emit_g = emit_g; p.emit_x = (bf16*)emit_x; p.emit_part = emit_part;
     p.split_flags = g_split_flags;
     p.act_limit = act_limit;
+    p.squared_relu = relu2 ? 1 : 0;
     dim3 grid((N + BM - 1) / BM, (T + pl.bn - 1) / pl.bn, pl.splits);
     if (grid.y > 65535) return CW_ERR_BAD_SIZE;
     if (pl.pair) {

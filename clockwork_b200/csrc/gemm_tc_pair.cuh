@@ -281,7 +281,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
                 asm volatile("bar.sync 2, 128;" ::: "memory");
 #pragma unroll
                 for (int j = 0; j < 16; ++j) {
-                    const float v = g[j] + bias;
+                    float v = g[j] + bias;
+                    if (!SWIGLU && p.squared_relu) v = squared_relu(v);
                     if (wide)
                         st32[j * BM + row] = v;
                     else

@@ -22,6 +22,8 @@
 #define GG_EPI_STORE_F32 1    // C (float) = acc
 #define GG_EPI_SILU_MUL 2     // C (T) = silu(acc) * acc2, acc2 from B2; with a positive `glu_limit` the clamped form below
 #define GG_EPI_SIGMOID_GATE 3 // C (T) = acc * sigmoid(gate[dst, c_group_off*g + n])
+#define GG_EPI_RELU2 4        // C (T) = max(acc, 0)^2
+#define GG_EPI_GROUP_GATE 5   // C (T) = acc * sigmoid(gate[dst, g]), `gate` float32: one number per row and group
 
 // The gated activation of the two-product form: silu(a) b, or, with a positive limit,
 //   a' = min(a, limit), b' = clamp(b, -limit, limit):  a' sigmoid(1.702 a') (b' + 1)
@@ -129,6 +131,8 @@ grouped_gemm_kernel(const T* __restrict__ A, int lda, int a_group_off, const T* 
             } else {
                 if (EPI == GG_EPI_SILU_MUL) v = gg_glu(v, acc2[r][c], glu_limit);
                 if (EPI == GG_EPI_SIGMOID_GATE) v = v / (1.f + expf(-to_f(gate[(size_t)d * ldg + (size_t)g * c_group_off + n])));
+                if (EPI == GG_EPI_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
+                if (EPI == GG_EPI_GROUP_GATE) v = v / (1.f + expf(-((const float*)gate)[(size_t)d * ldg + g]));
                 ((T*)Cv)[at] = from_f<T>(v);
             }
         }
@@ -279,6 +283,7 @@ grouped_gemm_mma_kernel(const bf16* __restrict__ A, int lda, int a_group_off, co
         for (int half = 0; half < 2; ++half) {
             const int d = dst_s[wm * 32 + mi * 16 + half * 8 + (lane >> 2)];
             if (d < 0) continue;
+            const float open = EPI == GG_EPI_GROUP_GATE ? 1.f / (1.f + expf(-((const float*)gate)[(size_t)d * ldg + g])) : 1.f;
 #pragma unroll
             for (int ni = 0; ni < 4; ++ni) {
 #pragma unroll
@@ -293,6 +298,8 @@ grouped_gemm_mma_kernel(const bf16* __restrict__ A, int lda, int a_group_off, co
                         if (TWO) v = gg_glu(v, acc2[TWO ? mi : 0][TWO ? ni : 0][half * 2 + e], glu_limit);
                         if (EPI == GG_EPI_SIGMOID_GATE)
                             v = v / (1.f + expf(-to_f(gate[(size_t)d * ldg + (size_t)g * c_group_off + n])));
+                        if (EPI == GG_EPI_RELU2) v = fmaxf(v, 0.f) * fmaxf(v, 0.f);
+                        if (EPI == GG_EPI_GROUP_GATE) v *= open;
                         ((bf16*)Cv)[at] = __float2bfloat16_rn(v);
                     }
                 }
@@ -334,6 +341,8 @@ static int launch_grouped(int epi, dim3 grid, cudaStream_t stream, const void* A
         case GG_EPI_STORE_F32: GG_GO(GG_EPI_STORE_F32);
         case GG_EPI_SILU_MUL: GG_GO(GG_EPI_SILU_MUL);
         case GG_EPI_SIGMOID_GATE: GG_GO(GG_EPI_SIGMOID_GATE);
+        case GG_EPI_RELU2: GG_GO(GG_EPI_RELU2);
+        case GG_EPI_GROUP_GATE: GG_GO(GG_EPI_GROUP_GATE);
     }
 #undef GG_GO
     return CW_ERR_UNSUPPORTED;
@@ -349,7 +358,7 @@ extern "C" int cw_grouped_gemm(const void* A, int lda, int a_group_off, const vo
     if (M == 0) return CW_OK;
     if (M < 0 || Nout <= 0 || K <= 0 || G <= 0 || a_div <= 0) return CW_ERR_BAD_SIZE;
     if (epilogue == GG_EPI_SILU_MUL && B2 == nullptr) return CW_ERR_BAD_SIZE;
-    if (epilogue == GG_EPI_SIGMOID_GATE && gate == nullptr) return CW_ERR_BAD_SIZE;
+    if ((epilogue == GG_EPI_SIGMOID_GATE || epilogue == GG_EPI_GROUP_GATE) && gate == nullptr) return CW_ERR_BAD_SIZE;
     const long long tiles = offsets == nullptr ? (long long)G * ((M + GG_TM - 1) / GG_TM) : (long long)(M + GG_TM - 1) / GG_TM + G;
     if (tiles > 0x7fffffffLL) return CW_ERR_UNSUPPORTED;
     dim3 grid((unsigned)tiles, (Nout + GG_TN - 1) / GG_TN);
@@ -369,6 +378,8 @@ extern "C" int cw_grouped_gemm(const void* A, int lda, int a_group_off, const vo
             case GG_EPI_STORE_F32: GM_GO(GG_EPI_STORE_F32);
             case GG_EPI_SILU_MUL: GM_GO(GG_EPI_SILU_MUL);
             case GG_EPI_SIGMOID_GATE: GM_GO(GG_EPI_SIGMOID_GATE);
+            case GG_EPI_RELU2: GM_GO(GG_EPI_RELU2);
+            case GG_EPI_GROUP_GATE: GM_GO(GG_EPI_GROUP_GATE);
         }
 #undef GM_GO
         return CW_ERR_UNSUPPORTED;
@@ -383,17 +394,19 @@ extern "C" int cw_grouped_gemm(const void* A, int lda, int a_group_off, const vo
 // logits [N, E] float32 (a product with float32 accumulation, made by the caller) + bias; the `top`
 // largest (the lower index wins a tie).  sel < 0 marks a padding row.  A warp per token.
 //   mode 0: weights = softmax over the chosen logits.
-//   mode 1: scores = softmax over all E logits; weights = the chosen experts' scores as they are.
+//   mode 1: scores = softmax over all E logits; experts are ranked by score + correction[e] (`correction` null: by the
+//           score), weights = the chosen experts' scores without the correction.
 //   mode 2: scores = sigmoid of each logit; experts are ranked by score + correction[e] (`correction` null: by the score),
 //           weights = the chosen experts' scores without the correction.
-// Every weight is multiplied by weight_scale at the end.
+// `renormalize` (modes 1 and 2): the weights are divided by (their sum + 1e-20).  Every weight is multiplied by weight_scale
+// at the end.
 // groups > 1: the experts lie in `groups` equal runs of neighbours; a run counts as the sum of its `group_rank` largest
 // entries (1: its largest entry), and only experts of the `keep` best runs can be chosen (the others count as minus
 // infinity, whatever the sign of the entries).
 __global__ void __launch_bounds__(128)
 moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ b, const int* __restrict__ tok_seq,
                   int* __restrict__ sel, float* __restrict__ wt, int N, int E, int top, int mode, int groups, int keep,
-                  const float* __restrict__ correction, float weight_scale, int group_rank) {
+                  const float* __restrict__ correction, float weight_scale, int group_rank, int renormalize) {
     extern __shared__ float choose_s[];  // per warp: [E] logits or scores, [top] chosen ones, [groups] the runs' best, [E] plain scores
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -409,7 +422,7 @@ moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ b,
     float* logit_s = choose_s + (size_t)warp * (2 * E + top + groups);
     float* chosen_s = logit_s + E;
     float* group_s = chosen_s + top;
-    float* score_s = group_s + groups;  // mode 2: the scores that become weights
+    float* score_s = group_s + groups;  // modes 1 and 2: the scores that become weights
     for (int e = lane; e < E; e += 32) logit_s[e] = logits[(size_t)row * E + e] + (b != nullptr ? b[e] : 0.f);
     __syncwarp();
     if (mode == 1) {  // every expert's share of the softmax over all of them (sums in a fixed order)
@@ -419,7 +432,11 @@ moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ b,
         float sum = 0.f;
         for (int e = lane; e < E; e += 32) sum += expf(logit_s[e] - mx);
         sum = warp_sum(sum);
-        for (int e = lane; e < E; e += 32) logit_s[e] = expf(logit_s[e] - mx) / sum;
+        for (int e = lane; e < E; e += 32) {
+            const float sc = expf(logit_s[e] - mx) / sum;
+            score_s[e] = sc;
+            logit_s[e] = sc + (correction != nullptr ? correction[e] : 0.f);
+        }
         __syncwarp();
     }
     if (mode == 2) {
@@ -488,11 +505,13 @@ moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ b,
         }
         __syncwarp();
     }
-    if (mode == 1) {
-        for (int t = lane; t < top; t += 32) wt[(size_t)row * top + t] = chosen_s[t] == -INFINITY ? 0.f : chosen_s[t] * weight_scale;
-        return;
-    }
-    if (mode == 2) {
+    if (mode != 0) {
+        if (renormalize) {
+            float total = 0.f;
+            for (int t = 0; t < top; ++t)  // the same order in every lane
+                if (chosen_s[t] != -INFINITY) total += score_s[sel[(size_t)row * top + t]];
+            weight_scale /= total + 1e-20f;
+        }
         for (int t = lane; t < top; t += 32) {
             const int e = sel[(size_t)row * top + t];  // (written by lane 0 above, made visible by __syncwarp)
             wt[(size_t)row * top + t] = chosen_s[t] == -INFINITY ? 0.f : score_s[e] * weight_scale;
@@ -507,15 +526,16 @@ moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ b,
 
 extern "C" int cw_moe_choose(const float* logits, const float* b, const int* tok_seq, int* sel, float* wt, int N, int E, int top,
                              int mode, int groups, int keep, const float* correction, float weight_scale, int group_rank,
-                             cudaStream_t stream) {
+                             int renormalize, cudaStream_t stream) {
     if (N == 0) return CW_OK;
     if (N < 0 || E <= 0 || top <= 0 || top > E || mode < 0 || mode > 2) return CW_ERR_BAD_SIZE;
+    if (renormalize && mode == 0) return CW_ERR_BAD_SIZE;  // (already shares of the chosen ones)
     if (groups < 1 || E % groups || keep < 1 || keep > groups || (long long)keep * (E / groups) < top) return CW_ERR_BAD_SIZE;
     if (group_rank < 1 || group_rank > 4 || group_rank > E / groups) return CW_ERR_BAD_SIZE;
     const size_t smem = 4 * (size_t)(2 * E + top + groups) * sizeof(float);
     if (smem > (48 << 10)) return CW_ERR_UNSUPPORTED;
     return cw_launch_ordered(moe_choose_kernel, dim3((N + 3) / 4), dim3(128), smem, stream, logits, b, tok_seq, sel, wt, N, E, top,
-                             mode, groups, keep, correction, weight_scale, group_rank);
+                             mode, groups, keep, correction, weight_scale, group_rank, renormalize);
 }
 
 // ---- pairs by expert --------------------------------------------------------------------------------
@@ -557,10 +577,11 @@ extern "C" int cw_moe_group(const int* sel, int* offsets, int* order, int* rank,
 }
 
 // resid[n] += sum_t wt[n, t] * y[n * top + t] over the choices in order; with `assign` the sum replaces resid[n] (rows of no
-// request: zeros).
+// request: zeros).  A choice of `experts` or above is an expert that hands its input on: x[n] stands in the place of its y.
+template <typename T>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(float* __restrict__ resid, const float* __restrict__ y, const int* __restrict__ sel,
-                   const float* __restrict__ wt, int W, int top, int assign) {
+                   const float* __restrict__ wt, const T* __restrict__ x, int experts, int W, int top, int assign) {
     pdl_wait();
     const int row = blockIdx.x;
     if (sel[(size_t)row * top] < 0) {
@@ -570,16 +591,24 @@ moe_combine_kernel(float* __restrict__ resid, const float* __restrict__ y, const
     }
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         float acc = 0.f;
-        for (int t = 0; t < top; ++t) acc = fmaf(wt[(size_t)row * top + t], y[((size_t)row * top + t) * W + c], acc);
+        for (int t = 0; t < top; ++t) {
+            const bool kept = x != nullptr && sel[(size_t)row * top + t] >= experts;
+            acc = fmaf(wt[(size_t)row * top + t], kept ? to_f(x[(size_t)row * W + c]) : y[((size_t)row * top + t) * W + c], acc);
+        }
         resid[(size_t)row * W + c] = assign ? acc : resid[(size_t)row * W + c] + acc;
     }
 }
 
-extern "C" int cw_moe_combine(float* resid, const float* y, const int* sel, const float* wt, int N, int W, int top, int assign,
-                              cudaStream_t stream) {
+// x null: every choice below `experts` (whatever it is) has its y.  dtype: of x.
+extern "C" int cw_moe_combine(float* resid, const float* y, const int* sel, const float* wt, const void* x, int experts, int N,
+                              int W, int top, int assign, int dtype, cudaStream_t stream) {
     if (N == 0) return CW_OK;
-    if (N < 0 || W <= 0 || top <= 0) return CW_ERR_BAD_SIZE;
-    return cw_launch_ordered(moe_combine_kernel, dim3(N), dim3(256), 0, stream, resid, y, sel, wt, W, top, assign);
+    if (N < 0 || W <= 0 || top <= 0 || (x != nullptr && experts < 0)) return CW_ERR_BAD_SIZE;
+    if (dtype == 0)
+        return cw_launch_ordered(moe_combine_kernel<float>, dim3(N), dim3(256), 0, stream, resid, y, sel, wt, (const float*)x, experts, W, top, assign);
+    if (dtype == 1)
+        return cw_launch_ordered(moe_combine_kernel<bf16>, dim3(N), dim3(256), 0, stream, resid, y, sel, wt, (const bf16*)x, experts, W, top, assign);
+    return CW_ERR_BAD_DTYPE;
 }
 
 CW_TRACE_TU(grouped_gemm)

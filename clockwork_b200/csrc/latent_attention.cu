@@ -8,29 +8,32 @@
 // so a query row is [W_uk,h^T q_plain | q_rot] (rank + rot numbers per head, made by a grouped product
 // and cw_latent_prepare), all heads read the same cached rows, and the kernel returns sum_j p c_j per
 // head for another grouped product to map to the head's value size.  The sink is a learned number per
-// head that takes part in the softmax denominator only (no key, no value, not scaled, counted once).
+// head that takes part in the softmax denominator only (no key, no value, not scaled, counted once; a layer may have none).
 //
-//   cw_latent_prepare    RMS norm of the latent (float32) and rotation of the shared key part, written to
+//   cw_latent_prepare    RMS norm of the latent (float32) and rotation of the shared key part (rotation.cuh), written to
 //                        the cache row of the token's slot; rotation of the queries' rotated parts
 //   cw_latent_attention  causal attention of a flat batch (prompt portions beside single tokens) over the
 //                        paged rows; float32 scores, weights and accumulation in both run precisions
-#include "common.cuh"
+#include "rotation.cuh"
 
-// down [N, rank + rot] float32 (the projection's output), q [N, H*(dim+rot)], qa [N, H*(rank+rot)] (the
-// rotated parts are written at [.., rank:]), cache [slots, rank + rot].  Pair (i, i + rot/2) at position p
-// turns by the angle p * inv_freq[i].
-template <typename T>
-__global__ void __launch_bounds__(128)
-latent_prepare_kernel(const float* __restrict__ down, const T* __restrict__ q, T* __restrict__ qa, T* __restrict__ cache,
-                      const float* __restrict__ norm_w, const float* __restrict__ inv_freq,
-                      const int* __restrict__ positions, const int* __restrict__ slots, int H, int dim, int rot, int rank,
-                      int num_slots, float eps, int write_cache, int* status) {
+// down [N, rank + rot] (row stride ldd, float32: the projection's output); q [N, H*(dim + rot)] (row stride ldq, QT: float32
+// when one product made both, else T): per head [plain | rotated].  Written: the cache row [normed latent | rotated shared key
+// part] of the token's slot, the queries' rotated parts into qa [N, H*(rank+rot)] at [.., rank:] of every head and, with
+// q_plain [N, H*dim], their plain parts.
+template <typename T, typename QT>
+__global__ void __launch_bounds__(256)
+latent_prepare_kernel(const float* __restrict__ down, int ldd, const QT* __restrict__ q, int ldq, T* __restrict__ q_plain,
+                      T* __restrict__ qa, T* __restrict__ cache, const float* __restrict__ norm_w, Rotation rot,
+                      const int* __restrict__ positions, const int* __restrict__ slots, int H, int dim, int rank, int num_slots,
+                      float eps, int write_cache, int vec, int* status) {
+    extern __shared__ float lp_table[];  // cosines, then sines, of the token's pairs
     __shared__ float scratch[33];
     pdl_wait();
     const int row = blockIdx.x, tid = threadIdx.x;
-    const int D = rank + rot, half = rot / 2;
-    const float pos = (float)positions[row];
-    const float* dr = down + (size_t)row * D;
+    const int D = rank + rot.dims, half = rot.dims >> 1;
+    float *cs = lp_table, *sn = lp_table + half;
+    rotation_table(rot, positions[row], cs, sn);
+    const float* dr = down + (size_t)row * ldd;
     int slot = write_cache ? slots[row] : -1;
     if (slot >= num_slots) {
         if (tid == 0) cw_report(status, CW_ST_SLOT_RANGE, row, slot);
@@ -39,43 +42,66 @@ latent_prepare_kernel(const float* __restrict__ down, const T* __restrict__ q, T
     float ss = 0.f;
     for (int i = tid; i < rank; i += blockDim.x) ss = fmaf(dr[i], dr[i], ss);
     ss = block_sum(ss, scratch);
+    __syncthreads();  // the table is written
     const float inv = 1.0f / sqrtf(ss / (float)rank + eps);
     if (slot >= 0) {
         T* cr = cache + (size_t)slot * D;
         for (int i = tid; i < rank; i += blockDim.x) cr[i] = from_f<T>(dr[i] * inv * norm_w[i]);
         for (int i = tid; i < half; i += blockDim.x) {
-            float sn, cs;
-            sincosf(pos * inv_freq[i], &sn, &cs);
-            const float u = dr[rank + i], v = dr[rank + half + i];
-            cr[rank + i] = from_f<T>(u * cs - v * sn);
-            cr[rank + half + i] = from_f<T>(v * cs + u * sn);
+            const int a = rank + rotation_first(rot, i), b = rank + rotation_second(rot, i);
+            const float u = dr[a], v = dr[b];
+            cr[a] = from_f<T>(u * cs[i] - v * sn[i]);
+            cr[b] = from_f<T>(v * cs[i] + u * sn[i]);
         }
     }
+    const QT* qr = q + (size_t)row * ldq;
     for (int idx = tid; idx < H * half; idx += blockDim.x) {
-        const int h = idx / half, i = idx % half;
-        float sn, cs;
-        sincosf(pos * inv_freq[i], &sn, &cs);
-        const T* qr = q + (size_t)row * H * (dim + rot) + (size_t)h * (dim + rot) + dim;
-        const float u = to_f(qr[i]), v = to_f(qr[half + i]);
+        const int h = idx / half, i = idx - h * half;
+        const int a = rotation_first(rot, i), b = rotation_second(rot, i);
+        const QT* from = qr + (size_t)h * (dim + rot.dims) + dim;
+        const float u = to_f(from[a]), v = to_f(from[b]);
         T* o = qa + (size_t)row * H * D + (size_t)h * D + rank;
-        o[i] = from_f<T>(u * cs - v * sn);
-        o[half + i] = from_f<T>(v * cs + u * sn);
+        o[a] = from_f<T>(u * cs[i] - v * sn[i]);
+        o[b] = from_f<T>(v * cs[i] + u * sn[i]);
+    }
+    if (q_plain == nullptr) return;
+    T* qp = q_plain + (size_t)row * H * dim;
+    if (vec) {  // four entries at a time
+        const int quads = dim >> 2;
+        for (int idx = tid; idx < H * quads; idx += blockDim.x) {
+            const int h = idx / quads, i = (idx - h * quads) * 4;
+            Vec4<T>::store(qp + (size_t)h * dim + i, Vec4<QT>::load(qr + (size_t)h * (dim + rot.dims) + i));
+        }
+        return;
+    }
+    for (int idx = tid; idx < H * dim; idx += blockDim.x) {
+        const int h = idx / dim, i = idx - h * dim;
+        qp[idx] = from_f<T>(to_f(qr[(size_t)h * (dim + rot.dims) + i]));
     }
 }
 
-extern "C" int cw_latent_prepare(const float* down, const void* q, void* qa, void* cache, const float* norm_w,
-                                 const float* inv_freq, const int* positions, const int* slots, int N, int H, int dim, int rot,
-                                 int rank, int num_slots, float eps, int write_cache, int dtype, int* status,
-                                 cudaStream_t stream) {
+extern "C" int cw_latent_prepare(const float* down, int ldd, const void* q, int ldq, int q_float32, void* q_plain, void* qa, void* cache,
+                                 const float* norm_w, const float* inv_freq, int interleaved, float amplitude, const int* positions,
+                                 const int* slots, int N, int H, int dim, int rot_dims, int rank, int num_slots, float eps,
+                                 int write_cache, int dtype, int* status, cudaStream_t stream) {
     if (N == 0) return CW_OK;
-    if (N < 0 || H <= 0 || dim < 0 || rot < 0 || rot % 2 || rank <= 0) return CW_ERR_BAD_SIZE;
+    const Rotation rot = {inv_freq, rot_dims, interleaved, amplitude};
+    if (N < 0 || H <= 0 || dim < 0 || !rotation_ok(rot, rot_dims) || rank <= 0 || ldd < rank + rot_dims || ldq < H * (dim + rot_dims))
+        return CW_ERR_BAD_SIZE;
+    if (rot_dims > 8192) return CW_ERR_UNSUPPORTED;
+    if (dtype != 0 && dtype != 1) return CW_ERR_BAD_DTYPE;
+    const bool wide_q = q_float32 || dtype == 0;  // q's entries are float32
+    const int vec = dim % 4 == 0 && rot_dims % 4 == 0 && ldq % 4 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)q_plain & 15) == 0;
+    const dim3 grid(N), block(H * (dim + rot_dims) > 1024 ? 256 : 128);
+    const size_t smem = sizeof(float) * (size_t)rot_dims;
     if (dtype == 0)
-        return cw_launch_ordered(latent_prepare_kernel<float>, dim3(N), dim3(128), 0, stream, down, (const float*)q, (float*)qa,
-                         (float*)cache, norm_w, inv_freq, positions, slots, H, dim, rot, rank, num_slots, eps, write_cache, status);
-    if (dtype == 1)
-        return cw_launch_ordered(latent_prepare_kernel<bf16>, dim3(N), dim3(128), 0, stream, down, (const bf16*)q, (bf16*)qa,
-                         (bf16*)cache, norm_w, inv_freq, positions, slots, H, dim, rot, rank, num_slots, eps, write_cache, status);
-    return CW_ERR_BAD_DTYPE;
+        return cw_launch_ordered(latent_prepare_kernel<float, float>, grid, block, smem, stream, down, ldd, (const float*)q, ldq, (float*)q_plain,
+                                 (float*)qa, (float*)cache, norm_w, rot, positions, slots, H, dim, rank, num_slots, eps, write_cache, vec, status);
+    if (wide_q)
+        return cw_launch_ordered(latent_prepare_kernel<bf16, float>, grid, block, smem, stream, down, ldd, (const float*)q, ldq, (bf16*)q_plain,
+                                 (bf16*)qa, (bf16*)cache, norm_w, rot, positions, slots, H, dim, rank, num_slots, eps, write_cache, vec, status);
+    return cw_launch_ordered(latent_prepare_kernel<bf16, bf16>, grid, block, smem, stream, down, ldd, (const bf16*)q, ldq, (bf16*)q_plain,
+                             (bf16*)qa, (bf16*)cache, norm_w, rot, positions, slots, H, dim, rank, num_slots, eps, write_cache, vec, status);
 }
 
 // One block per (token, group of LA_HB heads).  Keys in chunks of 128, a thread per key for the scores

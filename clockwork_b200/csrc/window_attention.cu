@@ -25,7 +25,10 @@
 // seen as one key and value, read from the second cache (its rows come first in a row's order of keys); `softcap`: the
 // score (after the numbers per head) becomes cap tanh(score / cap); `slopes`: slope[h] (p - j) is taken off the (capped)
 // score; a query temperature: the score is multiplied by 1 + coef ln(floor((p + 1) / every) + 1) first of all; `gate`: head
-// h's output is multiplied by sigmoid(gate[n, h]).
+// h's output is multiplied by sigmoid(gate[n, h]), or (`gate_entries`) its entry c by sigmoid(gate[n, h*dv + c]).
+// Where a head's value begins within its row is a parameter (`voff`, dk by default).  A layer whose values are its keys
+// before the rotation keeps rows [key with its `voff` leading entries rotated | those entries unrotated]: the value, with
+// its entries in the order [rest | leading ones], is the row's tail from `voff` on, and what is not rotated is kept once.
 // bfloat16 calls run the tensor-core form further down when it takes the sizes; the CUDA-core kernel is the float32
 // path and the fallback.
 //
@@ -72,14 +75,15 @@ extern "C" int cw_store_rows(const void* src, int ld, int col0, int width, void*
 // [H*dk] and k_norm [G*dk] the queries are first divided by the root mean square (eps inside the root) of all H*dk of them
 // and multiplied by q_norm, the keys likewise over their G*dk entries.  Then the leading entries of every query and key
 // head are rotated, everything in float32.  Queries go to q_out [N, H*dk], the rows [key | value] to the cache row that
-// the token's slot names (slots null or < 0: nothing is stored).  Blocks: (token, share of its entries; each share forms
-// the norms' sums again).  VEC: four neighbouring entries at a time, 16-byte accesses (head sizes a multiple of 4 entries,
+// the token's slot names (slots null or < 0: nothing is stored).  `tied`: the product holds no values (src is [queries |
+// keys]); behind the rotated key the cache row holds the dv leading entries of the key as projected.
+// Blocks: (token, share of its entries; each share forms the norms' sums again).  VEC: four neighbouring entries at a time, 16-byte accesses (head sizes a multiple of 4 entries,
 // rotated ones of 4 or, with half pairs, of 8).
 template <typename T, bool NORM, bool VEC>
 __global__ void __launch_bounds__(256)
 rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict__ positions, const int* __restrict__ tok_seq,
                     const int* __restrict__ slots, Rotation rot, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
-                    float eps, int H, int G, int dk, int dv, T* __restrict__ q_out, T* __restrict__ cache, long long total_rows,
+                    float eps, int H, int G, int dk, int dv, int tied, T* __restrict__ q_out, T* __restrict__ cache, long long total_rows,
                     int* __restrict__ status) {
     extern __shared__ float rs_table[];  // cosines, then sines, of the token's pairs
     __shared__ float scratch[33];
@@ -87,6 +91,7 @@ rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict
     const int n = blockIdx.x;
     const int at = blockIdx.y * blockDim.x + threadIdx.x, step = gridDim.y * blockDim.x;
     const int HQ = H * dk, row = dk + dv, half = rot.dims >> 1;
+    const int src_row = tied ? dk : row, src_v = tied ? 0 : dk;  // a key/value head's entries in src, and its value's first
     T* qo = q_out + (size_t)n * HQ;
     if (tok_seq[n] < 0) {  // padding of a fixed-shape step
         for (int c = at; c < HQ; c += step) qo[c] = from_f<T>(0.f);
@@ -106,13 +111,13 @@ rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict
             const int quads = dk >> 2;
             for (int c = threadIdx.x; c < G * quads; c += blockDim.x) {
                 const int g = c / quads;
-                ks = square(Vec4<float>::load(kv + (size_t)g * row + (c - g * quads) * 4), ks);
+                ks = square(Vec4<float>::load(kv + (size_t)g * src_row + (c - g * quads) * 4), ks);
             }
         } else {
             for (int c = threadIdx.x; c < HQ; c += blockDim.x) qs = fmaf(x[c], x[c], qs);
             for (int g = 0; g < G; ++g)
                 for (int i = threadIdx.x; i < dk; i += blockDim.x) {
-                    const float k = kv[(size_t)g * row + i];
+                    const float k = kv[(size_t)g * src_row + i];
                     ks = fmaf(k, k, ks);
                 }
         }
@@ -185,26 +190,27 @@ rotate_store_kernel(const float* __restrict__ src, int ld, const int* __restrict
         const int quads = row >> 2;
         for (int c = at; c < G * quads; c += step) {
             const int g = c / quads, i = (c - g * quads) * 4;
-            const float* head = kv + (size_t)g * row;
+            const float* head = kv + (size_t)g * src_row;
             Vec4<T>::store(to + (size_t)g * row + i, i < dk ? entries(head, NORM ? k_norm + (size_t)g * dk : nullptr, k_inv, i)
-                                                            : Vec4<float>::load(head + i));
+                                                            : Vec4<float>::load(head + src_v + i - dk));
         }
         return;
     }
     for (int c = at; c < G * row; c += step) {
         const int g = c / row, i = c - g * row;
-        to[c] = from_f<T>(i < dk ? entry(kv + (size_t)g * row, NORM ? k_norm + (size_t)g * dk : nullptr, k_inv, i) : kv[c]);
+        const float* head = kv + (size_t)g * src_row;
+        to[c] = from_f<T>(i < dk ? entry(head, NORM ? k_norm + (size_t)g * dk : nullptr, k_inv, i) : head[src_v + i - dk]);
     }
 }
 
 extern "C" int cw_rotate_store(const float* src, int ld, const int* positions, const int* tok_seq, const int* slots,
                                const float* inv_freq, int rot_dims, int interleaved, float amplitude, const float* q_norm,
-                               const float* k_norm, float eps, int N, int H, int G, int dk, int dv, void* q_out, void* cache,
+                               const float* k_norm, float eps, int N, int H, int G, int dk, int dv, int tied, void* q_out, void* cache,
                                long long total_rows, int dtype, int* status, cudaStream_t stream) {
     if (N == 0) return CW_OK;
     const Rotation rot = {inv_freq, rot_dims, interleaved, amplitude};
-    if (N < 0 || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || !rotation_ok(rot, dk) || ld < H * dk + G * (dk + dv) || total_rows < 0 ||
-        (q_norm == nullptr) != (k_norm == nullptr))
+    if (N < 0 || H <= 0 || G <= 0 || dk <= 0 || dv < (tied ? 0 : 1) || (tied && dv > dk) || !rotation_ok(rot, dk) ||
+        ld < H * dk + G * (tied ? dk : dk + dv) || total_rows < 0 || (q_norm == nullptr) != (k_norm == nullptr))
         return CW_ERR_BAD_SIZE;
     if (rot_dims > 8192) return CW_ERR_UNSUPPORTED;
     auto whole = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
@@ -221,13 +227,13 @@ extern "C" int cw_rotate_store(const float* src, int ld, const int* positions, c
     if (dtype == 0) {
         const auto kernel = q_norm != nullptr ? (vec ? rotate_store_kernel<float, true, true> : rotate_store_kernel<float, true, false>)
                                               : (vec ? rotate_store_kernel<float, false, true> : rotate_store_kernel<float, false, false>);
-        return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv,
+        return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv, tied,
                                  (float*)q_out, (float*)cache, total_rows, status);
     }
     if (dtype == 1) {
         const auto kernel = q_norm != nullptr ? (vec ? rotate_store_kernel<bf16, true, true> : rotate_store_kernel<bf16, true, false>)
                                               : (vec ? rotate_store_kernel<bf16, false, true> : rotate_store_kernel<bf16, false, false>);
-        return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv,
+        return cw_launch_ordered(kernel, grid, block, smem, stream, src, ld, positions, tok_seq, slots, rot, q_norm, k_norm, eps, H, G, dk, dv, tied,
                                  (bf16*)q_out, (bf16*)cache, total_rows, status);
     }
     return CW_ERR_BAD_DTYPE;
@@ -341,6 +347,8 @@ struct WindowAttentionArgs {
     const int* pool_tables;   // [S, pool_max_blocks]
     int pool_max_blocks, pool_pages;
     int keep;                 // the sequence's first `keep` positions are seen by every later one
+    int voff;                 // where a head's value begins in its row (row width voff + dv; below dk: key and value overlap)
+    int gate_entries;         // 1: the gate has a number per output entry ([N, ldg], ldg >= H*dv) instead of one per head
 };
 
 // how many pooled blocks position p sees: those that end at or before p - window
@@ -361,7 +369,7 @@ window_attention_kernel(const WindowAttentionArgs a) {
     pdl_wait();
     const int n = blockIdx.x, part = blockIdx.y, tid = threadIdx.x;
     const int H = a.H, G = a.G, dk = a.dk, dv = a.dv, TK = a.tile;
-    const int HV = H * dv, per = H / G, row_width = dk + dv;
+    const int HV = H * dv, per = H / G, row_width = a.voff + dv;
     const int seq = a.tok_seq[n];
     T* out = (T*)a.out + (size_t)n * HV;
     float* partial = a.parts > 1 ? a.partial + ((size_t)n * a.parts + part) * (HV + 2 * H) : nullptr;
@@ -489,7 +497,7 @@ window_attention_kernel(const WindowAttentionArgs a) {
             const int col = tid + r * blockDim.x;
             if (col < HV) {
                 const int h = col / dv, c = col - h * dv;
-                const size_t voff = (size_t)(h / per) * row_width + dk + c;
+                const size_t voff = (size_t)(h / per) * row_width + a.voff + c;
                 const float* w = wt + h * TK;
                 float sum = a.sigmoid_weights ? acc[r] : acc[r] * alpha[h];
                 for (int j = 0; j < nk; ++j) {
@@ -515,7 +523,7 @@ window_attention_kernel(const WindowAttentionArgs a) {
             } else {
                 const float l = a.sigmoid_weights ? 1.f : lrun[col / dv];
                 float y = a.sigmoid_weights ? acc[r] : (l > 0.f ? acc[r] / l : 0.f);
-                if (a.gate != nullptr) y *= 1.f / (1.f + expf(-a.gate[(size_t)n * a.ldg + col / dv]));
+                if (a.gate != nullptr) y *= 1.f / (1.f + expf(-a.gate[(size_t)n * a.ldg + (a.gate_entries ? col : col / dv)]));
                 out[col] = from_f<T>(y);
             }
         }
@@ -532,7 +540,8 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 window_merge_kernel(const float* __restrict__ partial, const int* __restrict__ positions, const int* __restrict__ tok_seq,
                     int H, int dv, int window, int parts, int part_keys, int sigmoid_weights, int all_parts, int blocked,
-                    const float* __restrict__ sink, T* __restrict__ out, int pool, int keep, const float* __restrict__ gate, int ldg) {
+                    const float* __restrict__ sink, T* __restrict__ out, int pool, int keep, const float* __restrict__ gate, int ldg,
+                    int gate_entries) {
     __shared__ float factor[64];
     __shared__ float denominator;
     pdl_wait();
@@ -559,11 +568,12 @@ window_merge_kernel(const float* __restrict__ partial, const int* __restrict__ p
     }
     __syncthreads();
     const float l = denominator;
-    const float open = gate != nullptr ? 1.f / (1.f + expf(-gate[(size_t)n * ldg + h])) : 1.f;
+    float open = gate != nullptr && !gate_entries ? 1.f / (1.f + expf(-gate[(size_t)n * ldg + h])) : 1.f;
     for (int c = threadIdx.x; c < dv; c += blockDim.x) {
         const int col = h * dv + c;
         float sum = 0.f;
         for (int s = 0; s < used; ++s) sum = fmaf(factor[s], base[(size_t)s * stride + col], sum);
+        if (gate != nullptr && gate_entries) open = 1.f / (1.f + expf(-gate[(size_t)n * ldg + col]));
         out[(size_t)n * HV + col] = from_f<T>((l > 0.f ? sum / l : 0.f) * open);
     }
 }
@@ -616,6 +626,10 @@ __device__ __forceinline__ void wm_split(float x, float y, unsigned& hi, unsigne
     lo = *reinterpret_cast<const unsigned*>(&l);
 }
 
+// Row stride in shared memory of rows whose key and value overlap: the next odd number of 16-byte pieces, so that eight
+// rows of a matrix load fall into distinct banks.
+__host__ __device__ __forceinline__ int wm_joint_stride(int row_width) { return row_width % 16 == 0 ? row_width + 8 : row_width; }
+
 template <int DVMAX>
 __global__ void __launch_bounds__(DVMAX > 128 ? 256 : 512)
 window_attention_mma_kernel(const WindowMmaArgs args) {
@@ -625,7 +639,8 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
     pdl_wait();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nwarps = blockDim.x >> 5;
     const int H = a.H, G = a.G, dk = a.dk, dv = a.dv, per = H / G, GC = args.gc;
-    const int HV = H * dv, row_width = dk + dv;
+    const int HV = H * dv, row_width = a.voff + dv;
+    const bool joint = a.voff < dk;  // key and value of a row overlap: the row lies in shared memory as it is
     const int part = blockIdx.z;
     bf16* out = (bf16*)a.out;
     // rows of the flat batch that belong to no request (padding of a fixed-shape step) come out as zeros
@@ -678,10 +693,11 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
     const int hi = p0 + rows;                            // positions below hi
     // shared memory: Q [nwarps][16][dk+8], then per stage K [GC][32][dk+8] and V [GC][32][dv+8] (bfloat16), then with
     // talk the scores of all heads [H][16][40] and the mixing matrix [H][H] (float32)
-    const int qs = dk + 8, ks_ = dk + 8, vs_ = dv + 8;
+    // (joint rows: [GC][32][row + 8 or 0], the next odd number of 16-byte pieces, the value `voff` entries into it)
+    const int qs = dk + 8, ks_ = joint ? wm_joint_stride(row_width) : dk + 8, vs_ = joint ? ks_ : dv + 8;
     bf16* Qs = (bf16*)wm_smem;
     bf16* KV = Qs + (size_t)nwarps * 16 * qs;
-    const size_t stage_elems = (size_t)GC * WM_BN * (ks_ + vs_);
+    const size_t stage_elems = (size_t)GC * WM_BN * (joint ? ks_ : ks_ + vs_);
     float* Ss = (float*)(KV + (size_t)args.stages * stage_elems);
     float* Tm = Ss + (size_t)H * 16 * 40;
     const bool talk = a.talk != nullptr;
@@ -701,7 +717,7 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
     // A thread copies the same 16-byte piece (key/value head g, piece c of the row) of every `kstep`-th key of a tile, so
     // that what does not change from tile to tile is worked out once; pages are found by a shift when their size is a
     // power of two.
-    const int chunks_per_row = row_width / 8, kchunks = dk / 8;
+    const int chunks_per_row = row_width / 8, kchunks = joint ? chunks_per_row : dk / 8;
     const int pieces = GC * chunks_per_row;                     // 16-byte pieces per key
     const bool strided = blockDim.x % pieces == 0 || pieces % blockDim.x == 0;
     const int page_shift = (a.page_size & (a.page_size - 1)) == 0 ? 31 - __clz(a.page_size) : -1;
@@ -805,7 +821,7 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
         }
         __syncthreads();  // the tile has landed (and Q, at the first)
         const bf16* Kt = KV + (size_t)stage * stage_elems + (size_t)gl * WM_BN * ks_;
-        const bf16* Vt = KV + (size_t)stage * stage_elems + (size_t)GC * WM_BN * ks_ + (size_t)gl * WM_BN * vs_;
+        const bf16* Vt = joint ? Kt + a.voff : KV + (size_t)stage * stage_elems + (size_t)GC * WM_BN * ks_ + (size_t)gl * WM_BN * vs_;
         float s[WM_BN / 8][4];
 #pragma unroll
         for (int nt = 0; nt < WM_BN / 8; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
@@ -962,7 +978,16 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
             }
         } else {
             float inv = a.sigmoid_weights ? 1.f : (l_run[x] > 0.f ? 1.f / l_run[x] : 0.f);
-            if (a.gate != nullptr) inv *= 1.f / (1.f + __expf(-a.gate[n * a.ldg + h]));
+            if (a.gate != nullptr && !a.gate_entries) inv *= 1.f / (1.f + __expf(-a.gate[n * a.ldg + h]));
+            if (a.gate != nullptr && a.gate_entries) {
+                const float* gr = a.gate + n * a.ldg + (size_t)h * dv + cpair;
+#pragma unroll
+                for (int nt = 0; nt < DVMAX / 8; ++nt)
+                    if (nt < nvt) {
+                        o[nt][2 * x] /= 1.f + __expf(-gr[nt * 8]);
+                        o[nt][2 * x + 1] /= 1.f + __expf(-gr[nt * 8 + 1]);
+                    }
+            }
 #pragma unroll
             for (int nt = 0; nt < DVMAX / 8; ++nt)
                 if (nt < nvt)
@@ -978,7 +1003,8 @@ extern "C" int cw_window_attention_set_mma(int on) { g_window_mma = on ? 1 : 0; 
 static int window_attention_mma(const WindowAttentionArgs& base, const int* q_start, int S, int N, cudaStream_t stream, int* launched) {
     *launched = 0;
     const int H = base.H, G = base.G, dk = base.dk, dv = base.dv, per = H / G;
-    if (!g_window_mma || q_start == nullptr || dk % 16 || dv % 8 || dv > 256 || per > 16 || base.ldq % 8 || ((uintptr_t)base.q & 15) ||
+    const bool joint = base.voff < dk;
+    if (!g_window_mma || q_start == nullptr || dk % 16 || dv % 8 || base.voff % 8 || dv > 256 || per > 16 || base.ldq % 8 || ((uintptr_t)base.q & 15) ||
         ((uintptr_t)base.cache & 15))
         return 0;
     const int max_warps = dv > 128 ? 8 : 16;
@@ -992,7 +1018,7 @@ static int window_attention_mma(const WindowAttentionArgs& base, const int* q_st
     const int nwarps = gc * per;
     if (nwarps > max_warps) return 0;
     auto bytes = [&](int stages) {
-        return sizeof(bf16) * ((size_t)nwarps * 16 * (dk + 8) + (size_t)stages * gc * WM_BN * (dk + dv + 16)) +
+        return sizeof(bf16) * ((size_t)nwarps * 16 * (dk + 8) + (size_t)stages * gc * WM_BN * (joint ? wm_joint_stride(base.voff + dv) : dk + dv + 16)) +
                (base.talk != nullptr ? sizeof(float) * ((size_t)H * 16 * 40 + (size_t)H * H) : 0);
     };
     int stages = 2;
@@ -1026,9 +1052,10 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
                                    void* out, int parts, float* partial, const int* q_start, int S, int dtype, int* status,
                                    float softcap, const float* slopes, float temp_coef, int temp_every, const float* gate, int ldg,
                                    int pool, const void* pool_cache, const int* pool_tables, int pool_max_blocks, int pool_pages,
-                                   int keep, cudaStream_t stream) {
+                                   int keep, int voff, int gate_entries, cudaStream_t stream) {
     if (N == 0) return CW_OK;
-    if (softcap < 0.f || temp_every < 0 || pool < 0 || (gate != nullptr && ldg < H)) return CW_ERR_BAD_SIZE;
+    if (softcap < 0.f || temp_every < 0 || pool < 0 || (gate != nullptr && ldg < (gate_entries ? H * dv : H))) return CW_ERR_BAD_SIZE;
+    if (voff < 0 || voff + dv < dk) return CW_ERR_BAD_SIZE;
     if (pool > 0 && (pool_cache == nullptr || pool_tables == nullptr || pool_max_blocks <= 0 || pool_pages <= 0 || blocked || slopes != nullptr))
         return CW_ERR_BAD_SIZE;  // (a pooled block has no distance, and blocks of positions have nothing before them)
     if (keep < 0 || (keep > 0 && (blocked || pool > 0))) return CW_ERR_BAD_SIZE;  // (kept positions lie before a plain window)
@@ -1044,14 +1071,14 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
         const WindowAttentionArgs base = {q, ldq, cache, block_tables, max_blocks, page_size, num_pages, positions, tok_seq, H, G, dk, dv,
                                           window, scale, head_scale, talk, head_bias, sigmoid_weights, blocked, sink, out, WM_BN, parts, 0,
                                           partial, status, softcap, slopes, temp_coef, temp_every, gate, ldg, pool, pool_cache, pool_tables,
-                                          pool_max_blocks, pool_pages, keep};
+                                          pool_max_blocks, pool_pages, keep, voff, gate_entries};
         int launched = 0;
         const int rc = window_attention_mma(base, q_start, S, N, stream, &launched);
         if (rc != 0) return rc;
         if (launched) {
             if (parts == 1) return CW_OK;
             return cw_launch_ordered(window_merge_kernel<bf16>, dim3(N, H), dim3(merge_threads), 0, stream, (const float*)partial, positions, tok_seq, H,
-                                     dv, window, parts, 0, sigmoid_weights, 1, blocked, sink, (bf16*)out, pool, keep, gate, ldg);
+                                     dv, window, parts, 0, sigmoid_weights, 1, blocked, sink, (bf16*)out, pool, keep, gate, ldg, gate_entries);
         }
     }
     int threads = 128;
@@ -1073,7 +1100,7 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
     WindowAttentionArgs a = {q, ldq, cache, block_tables, max_blocks, page_size, num_pages, positions, tok_seq, H, G, dk, dv,
                              window, scale, head_scale, talk, head_bias, sigmoid_weights, blocked, sink, out, tile, parts, part_keys,
                              partial, status, softcap, slopes, temp_coef, temp_every, gate, ldg, pool, pool_cache, pool_tables,
-                             pool_max_blocks, pool_pages, keep};
+                             pool_max_blocks, pool_pages, keep, voff, gate_entries};
     static size_t allowed[2] = {48 << 10, 48 << 10};
     if (dtype != 0 && dtype != 1) return CW_ERR_BAD_DTYPE;
     if (smem > allowed[dtype]) {
@@ -1089,9 +1116,9 @@ extern "C" int cw_window_attention(const void* q, int ldq, const void* cache, co
     if (rc != 0 || parts == 1) return rc;
     if (dtype == 0)
         return cw_launch_ordered(window_merge_kernel<float>, dim3(N, H), dim3(merge_threads), 0, stream, (const float*)partial, positions, tok_seq,
-                                 H, dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (float*)out, pool, keep, gate, ldg);
+                                 H, dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (float*)out, pool, keep, gate, ldg, gate_entries);
     return cw_launch_ordered(window_merge_kernel<bf16>, dim3(N, H), dim3(merge_threads), 0, stream, (const float*)partial, positions, tok_seq, H,
-                             dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (bf16*)out, pool, keep, gate, ldg);
+                             dv, window, parts, part_keys, sigmoid_weights, 0, blocked, sink, (bf16*)out, pool, keep, gate, ldg, gate_entries);
 }
 
 CW_TRACE_TU(window_attention)

@@ -261,32 +261,38 @@ class PartialSums:
 
 
 def _add_partial_sums(resid: torch.Tensor, parts: PartialSums, weight: torch.Tensor | None, eps: float,
-                      out: torch.Tensor | None, center: bool = False) -> None:
+                      out: torch.Tensor | None, center: bool = False, weight2: torch.Tensor | None = None,
+                      out2: torch.Tensor | None = None) -> None:
     _need(parts.slabs, torch.float32, "partial sums", 3)
     n, h = resid.shape
     splits, slab_rows, width = parts.slabs.shape
     if width != h or parts.rows != n or slab_rows < n:
         raise ValueError(f"partial sums {tuple(parts.slabs.shape)} of {parts.rows} rows do not match residual {tuple(resid.shape)}")
     check(library().cw_add_parts_rmsnorm(_ptr(resid), _ptr(parts.slabs), splits, slab_rows, _ptr(weight), _ptr(out), n, h,
-                                         float(eps), 1 if center else 0, 0 if out is None else dtype_code(out.dtype), _stream()),
+                                         float(eps), 1 if center else 0, 0 if out is None else dtype_code(out.dtype), _ptr(weight2),
+                                         _ptr(out2), _stream()),
           "add_parts_rmsnorm")
 
 
 def add_rmsnorm(resid: torch.Tensor, delta, weight: torch.Tensor, eps: float,
-                out_dtype: torch.dtype, status: torch.Tensor, out: torch.Tensor | None = None, center: bool = False) -> torch.Tensor:
+                out_dtype: torch.dtype, status: torch.Tensor, out: torch.Tensor | None = None, center: bool = False,
+                weight2: torch.Tensor | None = None):
     """``resid += delta`` (if given: a tensor, or the ``PartialSums`` of a product), then returns
     ``weight * rmsnorm(resid)`` as ``out_dtype``.  ``center``: layer norm, the row's mean taken off first
-    (``(x - mean) / sqrt(mean of the squared deviations + eps) * weight``)."""
+    (``(x - mean) / sqrt(mean of the squared deviations + eps) * weight``).  ``weight2``: the pair of this and of the same
+    normalised rows times ``weight2``."""
     _need(resid, torch.float32, "resid", 2)
-    _need(weight, torch.float32, "weight", 1)
     n, h = resid.shape
-    if weight.shape[0] != h:
-        raise ValueError(f"norm weight has {weight.shape[0]} elements, rows have {h}")
+    for w in (weight,) if weight2 is None else (weight, weight2):
+        _need(w, torch.float32, "weight", 1)
+        if w.shape[0] != h:
+            raise ValueError(f"norm weight has {w.shape[0]} elements, rows have {h}")
+    out2 = None if weight2 is None else torch.empty((n, h), dtype=out_dtype, device=resid.device)
     if isinstance(delta, PartialSums):
         if out is None:
             out = torch.empty((n, h), dtype=out_dtype, device=resid.device)
-        _add_partial_sums(resid, delta, weight, eps, out, center)
-        return out
+        _add_partial_sums(resid, delta, weight, eps, out, center, weight2, out2)
+        return out if out2 is None else (out, out2)
     if delta is not None:
         _need(delta, out_dtype, "delta", 2)
         if delta.shape != resid.shape:
@@ -294,8 +300,9 @@ def add_rmsnorm(resid: torch.Tensor, delta, weight: torch.Tensor, eps: float,
     if out is None:
         out = torch.empty((n, h), dtype=out_dtype, device=resid.device)
     check(library().cw_add_rmsnorm(_ptr(resid), _ptr(delta), _ptr(weight), _ptr(out), None, n, n, h, float(eps),
-                                   1 if center else 0, dtype_code(out_dtype), _ptr(status), _stream()), "add_rmsnorm")
-    return out
+                                   1 if center else 0, dtype_code(out_dtype), _ptr(weight2), _ptr(out2), _ptr(status), _stream()),
+          "add_rmsnorm")
+    return out if out2 is None else (out, out2)
 
 
 def rmsnorm_rows(resid: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, eps: float,
@@ -308,7 +315,7 @@ def rmsnorm_rows(resid: torch.Tensor, rows: torch.Tensor, weight: torch.Tensor, 
     r = rows.shape[0]
     out = torch.empty((r, h), dtype=out_dtype, device=resid.device)
     check(library().cw_add_rmsnorm(_ptr(resid), None, _ptr(weight), _ptr(out), _ptr(rows), r, n, h, float(eps),
-                                   1 if center else 0, dtype_code(out_dtype), _ptr(status), _stream()), "rmsnorm_rows")
+                                   1 if center else 0, dtype_code(out_dtype), None, None, _ptr(status), _stream()), "rmsnorm_rows")
     return out
 
 
@@ -335,13 +342,14 @@ def add_to_residual(resid: torch.Tensor, delta) -> None:
 
 
 EPILOGUE_STORE, EPILOGUE_ADD_F32, EPILOGUE_STORE_F32 = 0, 1, 2
+EPILOGUE_RELU2 = 4  # store max(v, 0)^2 of v = product + bias, in the operands' dtype
 
 
 def gemm_ref(a: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, *,
              out: torch.Tensor | None = None, epilogue: int = EPILOGUE_STORE) -> torch.Tensor:
     """``a [M,K] @ w[N,K]^T (+ bias)`` on the CUDA cores with float32 accumulation.
     ``a`` may be a column slice of a wider matrix (row stride > K).  Epilogues: store in
-    ``a``'s dtype; add into the float32 ``out``; store float32."""
+    ``a``'s dtype; add into the float32 ``out``; store float32; ``EPILOGUE_RELU2``."""
     if not a.is_cuda or a.dim() != 2 or a.stride(1) != 1:
         raise ValueError("a must be a 2-d CUDA tensor with unit column stride")
     _need(w, a.dtype, "w", 2)
@@ -353,7 +361,7 @@ def gemm_ref(a: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
         _need(bias, torch.float32, "bias", 1)
         if bias.shape[0] != n:
             raise ValueError("bias length does not match w's rows")
-    want = a.dtype if epilogue == EPILOGUE_STORE else torch.float32
+    want = a.dtype if epilogue in (EPILOGUE_STORE, EPILOGUE_RELU2) else torch.float32
     if out is None:
         if epilogue == EPILOGUE_ADD_F32:
             raise ValueError("the add epilogue needs an output to add into")

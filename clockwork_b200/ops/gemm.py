@@ -11,7 +11,7 @@ from typing import Callable
 
 import torch
 
-from . import EPILOGUE_ADD_F32, EPILOGUE_STORE, EPILOGUE_STORE_F32, gemm_ref, gemm_ref_swiglu
+from . import EPILOGUE_ADD_F32, EPILOGUE_RELU2, EPILOGUE_STORE, EPILOGUE_STORE_F32, gemm_ref, gemm_ref_swiglu
 
 _tc = None  # set by ops.gemm_tc (imported at the end of this module)
 
@@ -62,6 +62,13 @@ def linear(x, w: torch.Tensor, bias: torch.Tensor | None) -> torch.Tensor:
     if _use_tc(xt, w):
         return _tc.gemm(xt, w, bias, epilogue=EPILOGUE_STORE)
     return gemm_ref(xt, w, bias, epilogue=EPILOGUE_STORE)
+
+
+def linear_relu2(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None) -> torch.Tensor:
+    """``max(x W^T (+ bias), 0)^2`` in ``x``'s dtype, rounded once."""
+    if _use_tc(x, w):
+        return _tc.gemm(x, w, bias, epilogue=EPILOGUE_RELU2)
+    return gemm_ref(x, w, bias, epilogue=EPILOGUE_RELU2)
 
 
 def linear_add_into(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, residual: torch.Tensor,

@@ -11,7 +11,7 @@ from ctypes import POINTER, byref, c_float, c_int, c_longlong, c_void_p
 
 import torch
 
-from . import EPILOGUE_STORE, _need, _ptr, _stream, device_status, gemm as gemm_dispatch
+from . import EPILOGUE_RELU2, EPILOGUE_STORE, _need, _ptr, _stream, device_status, gemm as gemm_dispatch
 from .library import check, library
 
 _state: dict[int, dict] = {}
@@ -196,7 +196,7 @@ def gemm_partial_sums(x: torch.Tensor, w: torch.Tensor, splits: int):
 def gemm(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, *, out: torch.Tensor | None = None,
          epilogue: int = EPILOGUE_STORE, row_scale: tuple | None = None, emit: tuple | None = None) -> torch.Tensor:
     """``x [T,K] @ w[N,K]^T (+ bias)`` in bfloat16 on the tensor cores, float32 accumulation.
-    Epilogues as for ``gemm_ref``: store bfloat16, add into float32 ``out``, store float32.
+    Epilogues as for ``gemm_ref``: store bfloat16, add into float32 ``out``, store float32, store the squared relu.
 
     An RMSNorm between two products can be split over them (at most ``NORM_SPLIT_MAX_TOKENS`` rows).
     ``emit=(g, xg, parts)`` with the add epilogue: beside ``out += ...`` the kernel writes
@@ -210,7 +210,7 @@ def gemm(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None, *, 
         raise ValueError(f"inner sizes differ: x has K={k}, w has K={w.shape[1]}")
     if bias is not None:
         _need(bias, torch.float32, "bias", 1)
-    want = torch.bfloat16 if epilogue == EPILOGUE_STORE else torch.float32
+    want = torch.bfloat16 if epilogue in (EPILOGUE_STORE, EPILOGUE_RELU2) else torch.float32
     if out is None:
         if epilogue == 1:
             raise ValueError("the add epilogue needs an output to add into")

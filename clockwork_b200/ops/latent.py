@@ -16,23 +16,37 @@ def set_tensor_cores(on: bool) -> None:
 
 def latent_prepare(down: torch.Tensor, q: torch.Tensor, qa: torch.Tensor, view, norm_weight: torch.Tensor,
                    inv_freq: torch.Tensor, positions: torch.Tensor, heads: int, dim: int, rot: int, rank: int, eps: float,
-                   status: torch.Tensor) -> None:
+                   status: torch.Tensor, interleaved: bool = False, amplitude: float = 1.0,
+                   q_plain: torch.Tensor | None = None) -> None:
     """Writes each token's cache row [normed latent | rotated shared key part] at its slot and the rotated
-    parts of the queries into ``qa`` [N, heads*(rank+rot)] at [.., rank:] of every head."""
-    _need(down, torch.float32, "down", 2)
-    _need(q, None, "q", 2)
-    _need(qa, q.dtype, "qa", 2)
+    parts of the queries into ``qa`` [N, heads*(rank+rot)] at [.., rank:] of every head; with ``q_plain`` [N, heads*dim] the
+    queries' plain parts go there.  ``down`` float32 [N, >= rank+rot] and ``q`` [N, >= heads*(dim+rot)] (float32 or ``qa``'s
+    dtype) may be column slices of one product's rows.  Entry i of a rotated part pairs with entry i + rot/2, or
+    (``interleaved``) entry 2i with entry 2i + 1; sines and cosines are multiplied by ``amplitude``."""
+    for name, t, width in (("down", down, rank + rot), ("q", q, heads * (dim + rot))):
+        if t.dim() != 2 or t.stride(1) != 1 or t.shape[1] < width:
+            raise ValueError(f"{name} must be [N, >= {width}] with unit column stride")
+    _need(qa, None, "qa", 2)
     cache = view.k_cache
-    _need(cache, q.dtype, "cache", 4)
+    _need(cache, qa.dtype, "cache", 4)
+    _need(inv_freq, torch.float32, "inv_freq", 1)
     n = q.shape[0]
-    if down.shape[1] != rank + rot or q.shape[1] != heads * (dim + rot) or qa.shape[1] != heads * (rank + rot):
+    if down.dtype != torch.float32 or q.dtype not in (torch.float32, qa.dtype):
+        raise ValueError("down must be float32, q float32 or of the run's dtype")
+    if down.shape[0] != n or tuple(qa.shape) != (n, heads * (rank + rot)) or (rot and inv_freq.shape[0] * 2 != rot):
         raise ValueError("widths do not match the head count and sizes")
+    if q_plain is not None:
+        _need(q_plain, qa.dtype, "q_plain", 2)
+        if tuple(q_plain.shape) != (n, heads * dim):
+            raise ValueError(f"q_plain {tuple(q_plain.shape)} is not [{n}, {heads * dim}]")
     if cache.shape[2] * cache.shape[3] != rank + rot:
         raise ValueError("cache rows do not hold rank + rot numbers")
     write = bool(view.write)
-    check(library().cw_latent_prepare(_ptr(down), _ptr(q), _ptr(qa), _ptr(cache), _ptr(norm_weight), _ptr(inv_freq), _ptr(positions),
-                                      _ptr(view.slots), n, heads, dim, rot, rank, cache.shape[0] * cache.shape[1], float(eps),
-                                      1 if write else 0, dtype_code(q.dtype), _ptr(status), _stream()), "latent_prepare")
+    ld = lambda t: t.stride(0) if n > 1 else max(t.stride(0), t.shape[1])  # noqa: E731
+    check(library().cw_latent_prepare(_ptr(down), ld(down), _ptr(q), ld(q), 1 if q.dtype == torch.float32 else 0, _ptr(q_plain), _ptr(qa),
+                                      _ptr(cache), _ptr(norm_weight), _ptr(inv_freq), 1 if interleaved else 0, float(amplitude),
+                                      _ptr(positions), _ptr(view.slots), n, heads, dim, rot, rank, cache.shape[0] * cache.shape[1],
+                                      float(eps), 1 if write else 0, dtype_code(qa.dtype), _ptr(status), _stream()), "latent_prepare")
 
 
 def latent_attention(qa: torch.Tensor, view, ctx, sink: torch.Tensor | None, heads: int, rank: int, rot: int,

@@ -14,10 +14,10 @@ P, I, F, LL = c_void_p, c_int, c_float, c_longlong
 # name -> argument types (the stream is the last c_void_p of each)
 _SIGNATURES: dict[str, list] = {
     "cw_embed": [P, P, P, I, I, I, I, F, P, P],
-    "cw_add_rmsnorm": [P, P, P, P, P, I, I, I, F, I, I, P, P],
+    "cw_add_rmsnorm": [P, P, P, P, P, I, I, I, F, I, I, P, P, P, P],
     "cw_silu_mul": [P, P, I, I, I, P],
     "cw_add_to_residual": [P, P, I, I, I, P],
-    "cw_add_parts_rmsnorm": [P, P, I, I, P, P, I, I, F, I, I, P],
+    "cw_add_parts_rmsnorm": [P, P, I, I, P, P, I, I, F, I, I, P, P, P],
     "cw_gemm_ref": [P, P, P, P, I, I, I, I, I, I, I, P],
     "cw_gemm_ref_swiglu": [P, P, P, P, I, I, I, I, P],
     "cw_rope_store": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, P],
@@ -45,13 +45,13 @@ _SIGNATURES: dict[str, list] = {
     # contributions (csrc/embed_norm.cu)
     "cw_store_rows": [P, I, I, I, P, P, I, LL, I, P, P],
     "cw_window_attention": [P, I, P, P, I, I, I, P, P, I, I, I, I, I, I, F, P, P, P, I, I, P, P, I, P, P, I, I, P,
-                            F, P, F, I, P, I, I, P, P, I, I, I, P],
+                            F, P, F, I, P, I, I, P, P, I, I, I, I, I, P],
     "cw_pool_rows": [P, P, I, I, I, P, P, P, P, LL, I, I, I, I, P, P],
     "cw_pair_embed_add": [P, P, P, P, P, P, P, LL, P, I, LL, LL, I, I, I, I, I, P, P],
     "cw_axpy_rmsnorm": [P, P, P, F, F, P, P, P, F, I, I, I, P],
     "cw_depth_average": [P, P, P, F, F, P, LL, I, P, P, P, P, F, I, I, I, P],
     "cw_bounded_forget": [P, I, P, P, P, I, I, P],
-    "cw_rotate_store": [P, I, P, P, P, P, I, I, F, P, P, F, I, I, I, I, I, P, P, LL, I, P, P],
+    "cw_rotate_store": [P, I, P, P, P, P, I, I, F, P, P, F, I, I, I, I, I, I, P, P, LL, I, P, P],
     "cw_window_attention_set_mma": [I],
     "cw_scale_add_sinusoid": [P, P, P, F, I, I, P],
     "cw_pair_rmsnorm_add": [P, P, P, P, P, F, F, I, I, P],
@@ -61,9 +61,9 @@ _SIGNATURES: dict[str, list] = {
     "cw_grouped_gemm": [P, I, I, P, P, LL, P, I, I, P, P, I, P, P, I, I, I, I, I, I, F, I, P],
     "cw_grouped_gemm_set_mma": [I],
     "cw_latent_attention_set_mma": [I],
-    "cw_moe_choose": [P, P, P, P, P, I, I, I, I, I, I, P, F, I, P],
+    "cw_moe_choose": [P, P, P, P, P, I, I, I, I, I, I, P, F, I, I, P],
     "cw_moe_group": [P, P, P, P, I, I, P],
-    "cw_moe_combine": [P, P, P, P, I, I, I, I, P],
+    "cw_moe_combine": [P, P, P, P, P, I, I, I, I, I, I, P],
     # the delta rule, the gates and the read-out of a matrix memory (csrc/recurrence_gated.cu)
     "cw_unit_heads": [P, I, I, I, I, F, I, F, F, P],
     "cw_delta_coefficients": [P, I, P, P, P, I, I, I, I, P],
@@ -72,7 +72,7 @@ _SIGNATURES: dict[str, list] = {
     "cw_gate_scan": [P, I, P, I, P, P, F, P, LL, LL, P, P, P, I, I, I, P, P],
     "cw_memory_norm": [P, P, I, P, I, P, P, I, I, I, F, I, P],
     # attention over a cached latent (csrc/latent_attention.cu)
-    "cw_latent_prepare": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P, P],
+    "cw_latent_prepare": [P, I, P, I, I, P, P, P, P, P, I, F, P, P, I, I, I, I, I, I, F, I, I, P, P],
     "cw_latent_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P],
 }
 _OPTIONAL: dict[str, list] = {}

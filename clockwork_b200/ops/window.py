@@ -48,14 +48,15 @@ def store_rows(src: torch.Tensor, col0: int, width: int, cache_rows: torch.Tenso
 
 def rotate_store(src: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tensor, slots: torch.Tensor | None, inv_freq: torch.Tensor | None,
                  heads: int, kv_heads: int, dk: int, dv: int, rot: int, cache_rows: torch.Tensor, status: torch.Tensor,
-                 interleaved: bool = False, amplitude: float = 1.0, norms: tuple | None = None) -> torch.Tensor:
+                 interleaved: bool = False, amplitude: float = 1.0, norms: tuple | None = None, tied: bool = False) -> torch.Tensor:
     """From the float32 product rows ``src`` [N, >= heads*dk + kv_heads*(dk + dv)] (queries, then ``[key | value]`` per
     key/value head): the first ``rot`` entries of every query and key head turned by the token's position (entry i with
     entry i + rot/2, or ``interleaved`` entry 2i with entry 2i + 1, by ``position * inv_freq[i]``, float32 angles, sines and
     cosines times ``amplitude``); returns the queries [N, heads*dk] in the cache's dtype and stores the rows
     ``[key | value]`` where ``slots`` says (None: nothing is stored).  ``norms`` = (query weight [heads*dk], key weight
     [kv_heads*dk], eps): first of all the token's queries, all heads together, are divided by their root mean square and
-    multiplied by the weight, and its keys likewise."""
+    multiplied by the weight, and its keys likewise.  ``tied``: ``src`` holds no values ([queries | keys]); behind the rotated
+    key a cache row holds the ``dv`` leading entries of the key as projected."""
     if src.dtype != torch.float32 or src.dim() != 2 or src.stride(1) != 1:
         raise ValueError("src must be float32 [N, C] with unit column stride")
     _need(cache_rows, None, "cache", 4)
@@ -76,7 +77,7 @@ def rotate_store(src: torch.Tensor, positions: torch.Tensor, tok_seq: torch.Tens
     total = cache_rows.shape[0] * cache_rows.shape[1]
     check(library().cw_rotate_store(_ptr(src), src.stride(0) if n > 1 else max(src.stride(0), src.shape[1]), _ptr(positions), _ptr(tok_seq),
                                     _ptr(slots), _ptr(inv_freq) if rot else None, rot, 1 if interleaved else 0, float(amplitude),
-                                    _ptr(q_norm), _ptr(k_norm), float(eps), n, heads, kv_heads, dk, dv, _ptr(q), _ptr(cache_rows),
+                                    _ptr(q_norm), _ptr(k_norm), float(eps), n, heads, kv_heads, dk, dv, 1 if tied else 0, _ptr(q), _ptr(cache_rows),
                                     total, dtype_code(cache_rows.dtype), _ptr(status), _stream()), "rotate_store")
     return q
 
@@ -129,7 +130,7 @@ def window_attention(q: torch.Tensor, cache_rows: torch.Tensor, block_tables: to
                      sink: torch.Tensor | None = None, softcap: float = 0.0, slopes: torch.Tensor | None = None,
                      temperature: tuple | None = None, gate: torch.Tensor | None = None, pool: int = 0,
                      pool_rows_cache: torch.Tensor | None = None, pool_tables: torch.Tensor | None = None,
-                     keep_first: int = 0) -> torch.Tensor:
+                     keep_first: int = 0, value_offset: int | None = None, gate_entries: bool = False) -> torch.Tensor:
     """[N, heads*dv] in ``q``'s dtype.  ``q`` [N, >= heads*dk] (queries in the leading columns, unit column stride);
     ``cache_rows`` [pages, page_size, kv_heads, dk + dv]; the step's tokens are already stored there.  ``blocked``:
     positions are cut into blocks of ``window`` and a token sees its own block up to itself, instead of the last
@@ -137,14 +138,17 @@ def window_attention(q: torch.Tensor, cache_rows: torch.Tensor, block_tables: to
     the score becomes ``softcap tanh(score / softcap)``; ``slopes`` [heads]: ``slopes[h] * (distance to the key)`` is taken
     off the (capped) score; ``temperature`` = (coef, every): the scores of a query at position p are first multiplied by
     ``1 + coef ln(floor((p + 1) / every) + 1)``; ``gate`` float32 [N, >= heads] (unit column stride): head h's output is
-    multiplied by ``sigmoid(gate[n, h])``; ``pool``: every block of ``pool`` positions that ends at or before p - window is
+    multiplied by ``sigmoid(gate[n, h])``, or with ``gate_entries`` (``gate`` [N, >= heads*dv]) every entry by the sigmoid of its
+    own number; ``value_offset``: where a head's value begins in its cache row (``dk`` when None), whose width is then
+    ``value_offset + dv``: below ``dk`` key and value overlap; ``pool``: every block of ``pool`` positions that ends at or before p - window is
     seen as one more key and value, row b of the request in ``pool_rows_cache`` (through ``pool_tables``); ``keep_first``:
     the sequence's first ``keep_first`` positions stay visible when the window has left them."""
     if q.dim() != 2 or q.stride(1) != 1 or q.shape[1] < heads * dk:
         raise ValueError("q must be [N, >= heads*dk] with unit column stride")
     _need(cache_rows, q.dtype, "cache", 4)
-    if tuple(cache_rows.shape[2:]) != (kv_heads, dk + dv):
-        raise ValueError(f"cache rows {tuple(cache_rows.shape)} are not [pages, page_size, {kv_heads}, {dk + dv}]")
+    voff = dk if value_offset is None else int(value_offset)
+    if tuple(cache_rows.shape[2:]) != (kv_heads, voff + dv):
+        raise ValueError(f"cache rows {tuple(cache_rows.shape)} are not [pages, page_size, {kv_heads}, {voff + dv}]")
     _need(block_tables, torch.int32, "block_tables", 2)
     _need(q_start, torch.int32, "q_start", 1)
     if sink is not None and sigmoid_weights:
@@ -160,8 +164,9 @@ def window_attention(q: torch.Tensor, cache_rows: torch.Tensor, block_tables: to
         _need(slopes, torch.float32, "slopes", 1)
         if slopes.shape[0] != heads:
             raise ValueError(f"slopes has {slopes.shape[0]} numbers for {heads} heads")
-    if gate is not None and (gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[1] < heads or gate.shape[0] != n):
-        raise ValueError("gate must be float32 [N, >= heads] with unit column stride")
+    gates = heads * dv if gate_entries else heads
+    if gate is not None and (gate.dtype != torch.float32 or gate.dim() != 2 or gate.stride(1) != 1 or gate.shape[1] < gates or gate.shape[0] != n):
+        raise ValueError(f"gate must be float32 [N, >= {gates}] with unit column stride")
     if pool:
         _need(pool_rows_cache, q.dtype, "pool cache", 4)
         _need(pool_tables, torch.int32, "pool_tables", 2)
@@ -182,5 +187,5 @@ def window_attention(q: torch.Tensor, cache_rows: torch.Tensor, block_tables: to
         _ptr(q_start), q_start.shape[0] - 1, dtype_code(q.dtype), _ptr(status),
         float(softcap), _ptr(slopes), float(coef), int(every), _ptr(gate), (gate.stride(0) if n > 1 else max(gate.stride(0), gate.shape[1])) if gate is not None else 0,
         int(pool), _ptr(pool_rows_cache) if pool else None, _ptr(pool_tables) if pool else None, pool_tables.shape[1] if pool else 0,
-        pool_rows_cache.shape[0] if pool else 0, int(keep_first), _stream()), "window_attention")
+        pool_rows_cache.shape[0] if pool else 0, int(keep_first), voff, 1 if gate_entries else 0, _stream()), "window_attention")
     return out

@@ -21,6 +21,10 @@ class Linear:
         """x [M, K] -> [M, N] in x's dtype."""
         return gemm_ops.linear(x, self.weight, self.bias)
 
+    def squared_relu(self, x: torch.Tensor) -> torch.Tensor:
+        """``max(x W^T (+ bias), 0)^2`` in x's dtype."""
+        return gemm_ops.linear_relu2(x, self.weight, self.bias)
+
     def add_into(self, x: torch.Tensor, residual: torch.Tensor, stream=None) -> None:
         """residual (float32 [M, N]) += x W^T (+ bias), the sum done in float32.  With the residual
         stream given, the product also begins the norm that the stream says comes next, when it can."""

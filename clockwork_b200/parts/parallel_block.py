@@ -1,8 +1,11 @@
-"""Parallel residual block: a single norm feeds the mixer and the feed-forward alike:
-``n = norm(h); h += mixer(n) + ffn(n)``.
+"""Parallel residual blocks: mixer and feed-forward read the same residual.
 
-Tensor prefixes: ``<layer>.norm1``, ``<layer>.mix``, ``<layer>.mlp`` (the names of the Rapitar
-checkpoints).  A layer without a feed-forward names the kind ``none``.  The sublayers' output
+``parallel_residual``: a single norm feeds both, ``n = norm(h); h += mixer(n) + ffn(n)``.
+``parallel_residual_two_norms``: each has a norm of its own, ``h += mixer(norm1(h)) + ffn(norm2(h))``; one kernel makes both
+norms in one pass over the rows.
+
+Tensor prefixes: ``<layer>.norm1`` (and ``<layer>.norm2``), ``<layer>.mix``, ``<layer>.mlp``.  A layer without a feed-forward
+names the kind ``none`` (and has no second norm).  The sublayers' output
 products add into the float32 residual in their epilogues, the mixer first, so the sum is
 ``(h + mixer) + ffn`` in float32 whatever the run precision.
 """
@@ -10,7 +13,7 @@ products add into the float32 residual in their epilogues, the mixer first, so t
 from __future__ import annotations
 
 from ..config.model_spec import LayerSpec
-from .base import Block, ResidualStream, StepContext
+from .base import Block, Norm, ResidualStream, StepContext
 from .registry import build_part, register_block
 
 
@@ -51,4 +54,50 @@ class ParallelResidualBlock(Block):
         stream.next_norm = None
 
 
+class NormPair(Norm):
+    """Two norms of the same rows as one part: ``forward`` returns both.  (It takes the slabs of a product whose splits are
+    kept apart like either of them, but no product can begin it: it has two weights.)"""
+
+    graph_safe = True
+    graph_safe_portions = True
+    takes_partial_sums = True
+
+    def __init__(self, first: Norm, second: Norm) -> None:
+        self.first, self.second = first, second
+
+    def tensor_decls(self):
+        yield from self.first.tensor_decls()
+        yield from self.second.tensor_decls()
+
+    def load_weights(self, fetch) -> None:
+        self.first.load_weights(fetch)
+        self.second.load_weights(fetch)
+
+    def forward(self, stream: ResidualStream, status, lazy: bool = False):
+        return self.first.forward_with(self.second, stream, status)
+
+
+class TwoNormParallelBlock(ParallelResidualBlock):
+    def __init__(self, layer: LayerSpec, dtype, device) -> None:
+        super().__init__(layer, dtype, device)
+        if self.ffn is not None:
+            second = build_part("norm", layer.ffn_norm, f"{layer.prefix}.norm2", dtype, device)
+            for norm in (self.norm, second):
+                if not hasattr(norm, "forward_with"):
+                    raise ValueError(f"norm kind {norm.spec.kind!r} cannot share a pass with another")
+            self.norm = NormPair(self.norm, second)
+
+    def forward(self, ctx: StepContext, stream: ResidualStream, view, following_norm=None) -> None:
+        if self.ffn is None:
+            super().forward(ctx, stream, view, following_norm)
+            return
+        x, y = self.norm.forward(stream, ctx.status)
+        stream.next_norm = None
+        stream.push(self.mixer.forward(ctx, x, view, stream))
+        stream.next_norm = following_norm
+        stream.push(self.ffn.forward(ctx, y, stream))
+        stream.next_norm = None
+
+
 register_block("parallel_residual", ParallelResidualBlock, replace=True)
+register_block("parallel_residual_two_norms", TwoNormParallelBlock, replace=True)

@@ -45,6 +45,15 @@ class WeightedNorm(Norm):
 
 
 class RMSNorm(WeightedNorm):
+    def forward_with(self, other: "RMSNorm", stream: ResidualStream, status: torch.Tensor) -> tuple:
+        """(this norm, ``other``) of the residual with what is pending added, in one pass over its rows: two norms that
+        differ in their weights only."""
+        if (other.size, other.eps) != (self.size, self.eps):
+            raise ValueError("norms that share a pass have the same size and eps")
+        stream.normed = stream.half_norm = None
+        delta, stream.pending = stream.pending, None
+        return ops.add_rmsnorm(stream.residual, delta, self.weight, self.eps, self.dtype, status, weight2=other.weight)
+
     def split_weight(self) -> torch.Tensor | None:
         """The weight a preceding product multiplies into the residual when it begins this norm."""
         return self.weight if self.dtype == torch.bfloat16 else None

@@ -21,6 +21,9 @@ Parameters: ``hidden_size, heads, kv_heads, dim`` (query/key size per head), ``v
 * ``distance_bias``: ``{"halvings": c}``: ``2^(-c (h + 1) / heads) * (t - j)`` is taken off head h's (capped) score;
 * ``query_temperature``: ``{"coef", "every"}``: the query at position t is multiplied by ``1 + coef ln(floor((t + 1) / every) + 1)``;
 * ``gate``: head h's output is multiplied by ``sigmoid(W_g x)_h`` before the output product (tensor ``g`` [heads, hidden]);
+  ``"entry"``: every entry of the heads' outputs by a sigmoid of its own (tensor ``g`` [heads*vdim, hidden]);
+* ``values``: ``"keys"``: there is no value product; the value of a key/value head is its key as projected, before the
+  rotation (``vdim`` = ``dim``; not together with ``pool``);
 * ``rotary``: ``{"dims", "base"}``: the first ``dims`` entries of every query and key head are rotated by the token's
   position before the key is cached, entry i with entry i + dims/2 by the angle ``t * base^(-2i/dims)`` (float32);
   ``"pairing": "interleaved"`` pairs entry 2i with entry 2i + 1 instead, ``"scaling"`` stretches the frequencies
@@ -39,7 +42,10 @@ whichever reaches farther back, since a block's mean is taken from the cached ro
 rows live in a page group of one row per ``pool`` positions, ``PagedKVNeed(every=pool)``).  At load the rows of k and v are
 interleaved head by head behind q, so that one product yields ``[q | k_0 v_0 | k_1 v_1 ..]`` per token and the
 cache write is a copy of the row's tail (with ``rotary`` the product's output is float32 and one kernel rotates,
-(and norms) rounds once and stores).  A blocked layer's page group gives back the pages of blocks that have passed.
+(and norms) rounds once and stores).  A layer whose values are its keys keeps ``[key, leading entries rotated | those entries
+unrotated]`` per token and key/value head, ``dim + rotary dims`` numbers: the value, with its entries in the order [rest |
+leading ones], is the row's tail, and the columns of ``o`` and the rows of an entry gate are put in that order at load.
+A blocked layer's page group gives back the pages of blocks that have passed.
 Scores, weights and weighted sums are float32 in either run precision.
 """
 
@@ -95,6 +101,12 @@ class WindowAttention(Mixer):
         if temp and self.temperature[1] < 1:
             raise ValueError("query_temperature.every must be at least 1")
         self.has_gate = bool(p.get("gate", False))
+        self.entry_gate = p.get("gate") == "entry"
+        self.tied = p.get("values") == "keys"
+        if p.get("values") not in (None, "keys"):
+            raise ValueError(f"values must be absent or 'keys', got {p.get('values')!r}")
+        if self.tied and (self.vdim != self.dim or self.pool):
+            raise ValueError("values that are the keys have the keys' size, and no pooled blocks")
         self.slopes = None
         self.keep_first = int(p.get("keep_first") or 0)
         if self.window >= window_ops.NO_WINDOW:
@@ -110,7 +122,11 @@ class WindowAttention(Mixer):
             raise ValueError(f"heads {self.heads} not a multiple of kv_heads {self.kv_heads}")
         if min(self.dim, self.vdim, self.window) <= 0:
             raise ValueError("dim, vdim and window must be positive")
-        self.row = self.dim + self.vdim
+        self.gates = 0 if not self.has_gate else self.heads * self.vdim if self.entry_gate else self.heads
+        # where a head's value begins in its cache row, and the row's width
+        self.value_offset = self.rot_dims if self.tied else self.dim
+        self.row = self.value_offset + self.vdim
+        self.kv_out = self.kv_heads * (self.dim if self.tied else self.row)  # columns of the product behind the queries
         self.qkv: Linear | None = None
         self.o: Linear | None = None
         self.head_scale = self.talk = self.head_bias = None
@@ -132,7 +148,8 @@ class WindowAttention(Mixer):
 
     def tensor_decls(self):
         h = self.hidden_size
-        for name, out in (("q", self.heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)):
+        products = [("q", self.heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
+        for name, out in products[:2] if self.tied else products:
             yield TensorDecl(self.name(name), (out, h), "matrix", "linear")
             if self.bias:
                 yield TensorDecl(self.name(f"{name}.b"), (out,), "vector", "bias")
@@ -148,7 +165,7 @@ class WindowAttention(Mixer):
         if self.has_sink and not self.zero_sink:
             yield TensorDecl(self.name("sink"), (self.heads,), "vector", "bias")
         if self.has_gate:
-            yield TensorDecl(self.name("g"), (self.heads, h), "matrix", "linear")
+            yield TensorDecl(self.name("g"), (self.gates, h), "matrix", "linear")
         yield TensorDecl(self.name("o"), (h, self.heads * self.vdim), "matrix", "linear")
         if self.out_bias:
             yield TensorDecl(self.name("o.b"), (h,), "vector", "bias")
@@ -159,18 +176,29 @@ class WindowAttention(Mixer):
         tail = k.shape[1:]
         return torch.cat([k.reshape(g, self.dim, *tail), v.reshape(g, self.vdim, *tail)], dim=1).reshape(g * self.row, *tail)
 
+    def _value_order(self, t: torch.Tensor) -> torch.Tensor:
+        """``t`` [heads*vdim, ..] with every head's entries in the order in which its output comes."""
+        if not self.tied or self.rot_dims in (0, self.dim):
+            return t
+        heads = t.reshape(self.heads, self.vdim, *t.shape[1:])
+        return torch.cat([heads[:, self.rot_dims :], heads[:, : self.rot_dims]], dim=1).reshape(t.shape)
+
     def load_weights(self, fetch) -> None:
-        q, k, v = (fetch(self.name(n)) for n in ("q", "k", "v"))
+        def by_kv_head(suffix: str) -> torch.Tensor:
+            k = fetch(self.name("k" + suffix))
+            return k if self.tied else self._rows_by_kv_head(k, fetch(self.name("v" + suffix)))
+
         # (with a gate its rows come last: one product yields [q | k_0 v_0 | .. | gate logits])
-        gate = [fetch(self.name("g"))] if self.has_gate else []
-        w = torch.cat([q, self._rows_by_kv_head(k, v), *gate], dim=0).contiguous()
+        gate = [] if not self.has_gate else [fetch(self.name("g"))]
+        if self.entry_gate:
+            gate = [self._value_order(gate[0])]
+        w = torch.cat([fetch(self.name("q")), by_kv_head(""), *gate], dim=0).contiguous()
         b = None
         if self.bias:
-            qb, kb, vb = (fetch(self.name(f"{n}.b")) for n in ("q", "k", "v"))
-            b = torch.cat([qb, self._rows_by_kv_head(kb, vb), *([torch.zeros_like(qb[: self.heads])] if self.has_gate else [])],
-                          dim=0).contiguous()
+            qb = fetch(self.name("q.b"))
+            b = torch.cat([qb, by_kv_head(".b"), torch.zeros(self.gates, dtype=qb.dtype, device=qb.device)], dim=0).contiguous()
         self.qkv = Linear(w, b)
-        self.o = Linear(fetch(self.name("o")), fetch(self.name("o.b")) if self.out_bias else None)
+        self.o = Linear(self._value_order(fetch(self.name("o")).T).T.contiguous(), fetch(self.name("o.b")) if self.out_bias else None)
         if self.has_head_scale:
             self.head_scale = fetch(self.name("temp")).contiguous()
         if self.has_talk:
@@ -192,16 +220,16 @@ class WindowAttention(Mixer):
         view, pooled = view if self.pool else (view, None)
         rows = view.k_cache  # [pages, page_size, kv_heads, dim + vdim]
         gate = None
-        if self.rot_dims or self.has_gate or self.qk_eps is not None:
+        if self.rot_dims or self.has_gate or self.qk_eps is not None or self.tied:
             # the product in float32, so that rotated queries and keys are rounded to the run's precision once (and the
             # gate's logits not at all)
             proj = self.qkv.to_float32(x)
             q = window_ops.rotate_store(proj, ctx.positions, ctx.tok_seq, view.slots if view.write else None,
-                                        self.inv_freq, self.heads, self.kv_heads, self.dim, self.vdim, self.rot_dims, rows, ctx.status,
-                                        self.interleaved, self.rot_amplitude,
-                                        None if self.qk_eps is None else (self.q_norm, self.k_norm, self.qk_eps))
+                                        self.inv_freq, self.heads, self.kv_heads, self.dim, self.row - self.dim, self.rot_dims, rows,
+                                        ctx.status, self.interleaved, self.rot_amplitude,
+                                        None if self.qk_eps is None else (self.q_norm, self.k_norm, self.qk_eps), self.tied)
             if self.has_gate:
-                gate = proj[:, self.heads * self.dim + self.kv_heads * self.row :]
+                gate = proj[:, self.heads * self.dim + self.kv_out :]
         else:
             q = self.qkv(x)  # [N, heads*dim | kv_heads*(dim + vdim)]
             if view.write:
@@ -215,7 +243,8 @@ class WindowAttention(Mixer):
                                            blocked=self.mask == "block", sink=self.sink, softcap=self.softcap, slopes=self.slopes,
                                            temperature=self.temperature, gate=gate, pool=self.pool,
                                            pool_rows_cache=pooled.k_cache if self.pool else None,
-                                           pool_tables=pooled.block_tables if self.pool else None, keep_first=self.keep_first)
+                                           pool_tables=pooled.block_tables if self.pool else None, keep_first=self.keep_first,
+                                           value_offset=self.value_offset, gate_entries=self.entry_gate)
 
     def mix(self, ctx: StepContext, x: torch.Tensor, view: PagedView) -> torch.Tensor:
         return self.o.to_float32(self._attend(ctx, x, view))
