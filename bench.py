@@ -382,8 +382,12 @@ def compare_designs(args) -> int:
     expert kernels).  With ``--design dezolorn`` the design is Dezolorn (``dezolorn-2k``: attention over a window of 1,024
     positions and the first 4, retention and delta-rule layers of 16 heads of 128 x 128, gated feed-forwards of 7,168, an output
     head of its own) beside Gamesun, the closest design the framework has (``gamesun-2k``: the same width, heads, layer
-    count and feed-forward; its layers run two mixers each, Dezolorn's one).  With ``--layers N`` both models have N layers.  One JSON
-    line; device time by CUDA events, medians."""
+    count and feed-forward; its layers run two mixers each, Dezolorn's one).  With ``--design relerax`` the design is Relerax
+    (``relerax-2k``: attention over a latent of 512 + 64 and over a window of 1,024 positions whose values are its keys, 16 heads
+    each, in turns; dense feed-forwards of 7,168 and 64 experts of 1,408 of which 6 are chosen, two norms a layer) beside
+    Rapitar, the closest design the framework has, with a layer list of the same width and count: latent attention of the
+    same heads, latent, key and value sizes in every layer, the same feed-forwards in the same places (``rapitar-latent-2k``).
+    With ``--layers N`` both models have N layers.  One JSON line; device time by CUDA events, medians."""
     import torch
 
     from clockwork_b200.cache import CacheManager
@@ -393,7 +397,7 @@ def compare_designs(args) -> int:
     assert torch.cuda.is_available(), "bench.py needs a CUDA device"
     torch.cuda.set_device(0)
     shape = {"rapitar": "rapitar-2k", "gamesun": "gamesun-2k", "kapolorn": "kapolorn-2k", "nuzulorn": "nuzulorn-2k",
-             "dezolorn": "dezolorn-2k"}[args.design]
+             "dezolorn": "dezolorn-2k", "relerax": "relerax-2k"}[args.design]
     rapitar = shape_config(shape, args.layers)
     layers = len(rapitar["layers"])
     qwen = dict(QWEN25_1P5B, num_hidden_layers=layers, hidden_size=2048, num_attention_heads=16,
@@ -407,6 +411,12 @@ def compare_designs(args) -> int:
         beside = ("gamesun-2k", shape_config("gamesun-2k", layers), rapitar["vocab"])
     if args.design == "nuzulorn":
         beside = ("kapolorn-2k", shape_config("kapolorn-2k", layers), rapitar["vocab"])
+    if args.design == "relerax":
+        closest = shape_config("rapitar-2k")
+        latent = next(layer["mixer"] for layer in closest["layers"] if layer["type"] == "latent_attention")
+        mlps = {kind: next(layer["mlp"] for layer in closest["layers"] if layer["mlp"]["kind"] == kind) for kind in ("dense", "moe")}
+        closest["layers"] = [{"type": "latent_attention", "mixer": latent, "mlp": mlps[layer["mlp"]["kind"]]} for layer in rapitar["layers"]]
+        beside = ("rapitar-latent-2k", closest, rapitar["vocab"])
     for name, raw, vocab in ((shape, rapitar, rapitar["vocab"]), beside):
         if args.model_filter and args.model_filter not in name:
             continue
@@ -474,7 +484,7 @@ def main() -> int:
     ap.add_argument("--top-k", type=int, default=-1)
     ap.add_argument("--top-p", type=float, default=1.0)
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the shape has (reported in config)")
-    ap.add_argument("--design", choices=["rapitar", "gamesun", "kapolorn", "nuzulorn", "dezolorn"], default="rapitar", help="with --only designs: which design stands beside Qwen2")
+    ap.add_argument("--design", choices=["rapitar", "gamesun", "kapolorn", "nuzulorn", "dezolorn", "relerax"], default="rapitar", help="with --only designs: which design stands beside Qwen2")
     ap.add_argument("--model-filter", default="", help="with --only designs: run only the model whose name holds this text (profiling runs)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--shape", default="qwen2.5-1.5b",

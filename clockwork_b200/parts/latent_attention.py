@@ -106,7 +106,7 @@ class LatentAttention(Mixer):
         self.sink = fetch(self.name("sink")) if self.has_sink else None
         self.o = Linear(fetch(self.name("o")))
 
-    def forward(self, ctx: StepContext, x, view: PagedView, stream: ResidualStream):
+    def _attend(self, ctx: StepContext, x, view: PagedView) -> torch.Tensor:
         n, heads, rank, rot = x.shape[0], self.heads, self.kv_rank, self.rot
         q_plain = head_gate = None
         if self.q_rank is not None:
@@ -132,7 +132,13 @@ class LatentAttention(Mixer):
         out = torch.empty((n, heads * self.vdim), dtype=self.dtype, device=x.device)
         grouped_ops.per_head_product(mixed, rank, self.uv, out, self.vdim,
                                      gate=self.gate(x) if self.gate_kind == "entry" else None, head_gate=head_gate)
-        return self.o.add_or_defer(out, stream)
+        return out
+
+    def mix(self, ctx: StepContext, x, view: PagedView) -> torch.Tensor:
+        return self.o.to_float32(self._attend(ctx, x, view))
+
+    def forward(self, ctx: StepContext, x, view: PagedView, stream: ResidualStream):
+        return self.o.add_or_defer(self._attend(ctx, x, view), stream)
 
 
 register_mixer("latent_attention", LatentAttention, replace=True)

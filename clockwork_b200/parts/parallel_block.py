@@ -13,6 +13,7 @@ products add into the float32 residual in their epilogues, the mixer first, so t
 from __future__ import annotations
 
 from ..config.model_spec import LayerSpec
+from ..weights.decl import TensorDecl
 from .base import Block, Norm, ResidualStream, StepContext
 from .registry import build_part, register_block
 
@@ -86,6 +87,11 @@ class TwoNormParallelBlock(ParallelResidualBlock):
                 if not hasattr(norm, "forward_with"):
                     raise ValueError(f"norm kind {norm.spec.kind!r} cannot share a pass with another")
             self.norm = NormPair(self.norm, second)
+
+    def tensor_decls(self):
+        yield from super().tensor_decls()
+        if self.ffn is None:  # (a checkpoint may hold the second norm all the same; nothing reads it)
+            yield TensorDecl(f"{self.prefix}.norm2", (int(self.layer.ffn_norm["size"]),), "vector", "norm", optional=True)
 
     def forward(self, ctx: StepContext, stream: ResidualStream, view, following_norm=None) -> None:
         if self.ffn is None:

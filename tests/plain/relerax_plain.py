@@ -151,7 +151,7 @@ def mixture(h, w, f, rnd=exact, margins=None):
     if margins is not None:
         margins.append(float(margin.min()))
     out = torch.zeros_like(h)
-    for e in range(f["router"]["experts"] + f["router"]["identity"]):
+    for e in range(w["router"].shape[0]):
         share = torch.where(chosen == e, weight, torch.zeros_like(weight)).sum(-1, keepdim=True)
         rows = share[:, 0] > 0
         if bool(rows.any()):
