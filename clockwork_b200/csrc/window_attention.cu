@@ -35,6 +35,7 @@
 // Scores, weights, the softmax statistics and the weighted sums are float32 in both run precisions; T names
 // the type of the product's output and of the cache.  A token's result depends on its position alone: keys
 // are taken in tiles that start at the window's first position, in order, whatever else the step holds.
+#include "request_tiles.cuh"
 #include "rotation.cuh"
 
 #define WA_MAX_COLS 16  // output columns per thread
@@ -651,23 +652,13 @@ window_attention_mma_kernel(const WindowMmaArgs args) {
                 for (int c = tid; c < HV; c += blockDim.x) out[(size_t)n * HV + c] = from_f<bf16>(0.f);
         }
     }
-    if (tid == 0) {  // which request and which 16 of its rows
-        int b = blockIdx.x, seq = -1, row0 = 0, rows = 0;
-        for (int s = 0; s < args.S; ++s) {
-            const int st = args.q_start[s], len = args.q_start[s + 1] - st;
-            if (len <= 0 || a.tok_seq[st] < 0) continue;
-            const int t = (len + 15) >> 4;
-            if (b < t) {
-                seq = s;
-                row0 = st + 16 * b;
-                rows = min(16, st + len - row0);
-                break;
-            }
-            b -= t;
+    if (warp == 0) {  // which request and which 16 of its rows
+        const RowTile tile = find_row_tile(blockIdx.x, false, args.q_start, a.tok_seq, args.S, 1, 16);
+        if (lane == 0) {
+            tile_seq = tile.seq;
+            tile_row0 = tile.row0;
+            tile_rows = tile.rows;
         }
-        tile_seq = seq;
-        tile_row0 = row0;
-        tile_rows = rows;
     }
     __syncthreads();
     const int seq = tile_seq, row0 = tile_row0, rows = tile_rows;

@@ -49,15 +49,52 @@ def latent_prepare(down: torch.Tensor, q: torch.Tensor, qa: torch.Tensor, view, 
                                       float(eps), 1 if write else 0, dtype_code(qa.dtype), _ptr(status), _stream()), "latent_prepare")
 
 
+MAX_PARTS = 128  # runs that a row's keys may be cut in
+TILE_ROWS = (16, 64)   # (token, head) rows per thread block: single tokens, portions
+FILL_BLOCKS = 148      # keys are cut until a step has about so many thread blocks (one to an SM)
+_scratch: dict[tuple, torch.Tensor] = {}  # (device index, rank) -> the partial sums of cut rows
+
+
+def _partial_sums(device, rank: int) -> torch.Tensor:
+    """Room for every step whose keys ``plan_parts`` cuts; made once and never replaced (captured steps point at it)."""
+    key = (torch.device(device).index or 0, rank)
+    have = _scratch.get(key)
+    if have is None:
+        have = _scratch[key] = torch.empty(FILL_BLOCKS * TILE_ROWS[1] * (rank + 2), dtype=torch.float32, device=device)
+    return have
+
+
+def reserve_scratch(device, rank: int, rot: int) -> None:
+    if library().cw_latent_attention_on_tensor_cores(rank, rot):
+        _partial_sums(device, rank)
+
+
+def plan_parts(tokens: int, seqs: int, heads: int, longest_portion: int, longest_context: int) -> tuple[bool, int]:
+    """(whether the step runs in tiles of few rows, in how many runs the keys of a row are cut): few rows over a long
+    context would otherwise leave most of the GPU idle.  What the device sees may be smaller than these bounds; a run
+    without keys costs a block that returns at once."""
+    few = longest_portion * heads <= 2 * TILE_ROWS[0]
+    if few and longest_portion <= 1:
+        tiles = seqs * -(-heads // TILE_ROWS[0])
+    else:
+        tiles = -(-tokens * heads // TILE_ROWS[0 if few else 1]) + seqs
+    return few, max(1, min(FILL_BLOCKS // max(1, tiles), -(-longest_context // 64), MAX_PARTS))
+
+
 def latent_attention(qa: torch.Tensor, view, ctx, sink: torch.Tensor | None, heads: int, rank: int, rot: int,
                      scale: float) -> torch.Tensor:
-    """[N, heads*rank]: per head the softmax-weighted sum of the cached latents (the sink in the denominator)."""
+    """[N, heads*rank]: per head the softmax-weighted sum of the cached latents (with a ``sink``, that in the denominator)."""
     _need(qa, None, "qa", 2)
+    _need(ctx.q_start, torch.int32, "q_start", 1)
     cache = view.k_cache
     n = qa.shape[0]
     out = torch.empty((n, heads * rank), dtype=qa.dtype, device=qa.device)
+    few, parts, partial = False, 1, None
+    if qa.dtype == torch.bfloat16 and library().cw_latent_attention_on_tensor_cores(rank, rot):
+        few, parts = plan_parts(n, ctx.num_seqs, heads, ctx.max_q_len, ctx.max_ctx_len)
+        partial = _partial_sums(qa.device, rank) if parts > 1 else None
     check(library().cw_latent_attention(_ptr(qa), _ptr(out), _ptr(cache), _ptr(view.block_tables), _ptr(ctx.tok_seq),
-                                        _ptr(ctx.positions), _ptr(sink), n, heads, rank, rot, cache.shape[1],
-                                        view.block_tables.shape[1], cache.shape[0], float(scale), dtype_code(qa.dtype),
-                                        _ptr(ctx.status), _stream()), "latent_attention")
+                                        _ptr(ctx.positions), _ptr(ctx.q_start), ctx.q_start.shape[0] - 1, _ptr(sink), n, heads, rank, rot,
+                                        cache.shape[1], view.block_tables.shape[1], cache.shape[0], float(scale), 1 if few else 0, parts,
+                                        _ptr(partial), dtype_code(qa.dtype), _ptr(ctx.status), _stream()), "latent_attention")
     return out

@@ -73,7 +73,8 @@ _SIGNATURES: dict[str, list] = {
     "cw_memory_norm": [P, P, I, P, I, P, P, I, I, I, F, I, P],
     # attention over a cached latent (csrc/latent_attention.cu)
     "cw_latent_prepare": [P, I, P, I, I, P, P, P, P, P, I, F, P, P, I, I, I, I, I, I, F, I, I, P, P],
-    "cw_latent_attention": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P],
+    "cw_latent_attention": [P, P, P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, I, I, P, I, P, P],
+    "cw_latent_attention_on_tensor_cores": [I, I],
 }
 _OPTIONAL: dict[str, list] = {}
 

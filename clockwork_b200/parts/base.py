@@ -255,11 +255,20 @@ class Mixer(Part):
 
 class FeedForward(Part):
     takes_half_normed = False
+    in_two_pieces = False  # True: ``begin`` and ``finish`` exist
 
     def output_terms(self, ctx: StepContext, x: torch.Tensor) -> list:
         """The feed-forward's output as one or two pairs (float32 [N, hidden], factor), added to nothing (see
         ``Mixer.mix_terms``).  Optional: only blocks that norm the output ask for it."""
         raise NotImplementedError(f"{type(self).__name__} cannot stand in a block that norms its output")
+
+    def begin(self, ctx: StepContext, x: torch.Tensor):
+        """What of ``forward`` does not touch the residual (for blocks that run it beside the mixer); ``finish`` is handed
+        the result.  Optional: a feed-forward without it runs in one piece."""
+        raise NotImplementedError(f"{type(self).__name__} does not run in two pieces")
+
+    def finish(self, ctx: StepContext, x: torch.Tensor, begun, stream: ResidualStream) -> torch.Tensor | None:
+        raise NotImplementedError(f"{type(self).__name__} does not run in two pieces")
 
     def forward(self, ctx: StepContext, x: torch.Tensor, stream: ResidualStream) -> torch.Tensor | None:
         raise NotImplementedError

@@ -95,8 +95,16 @@ class SquaredReluMLP(FeedForward):
     def load_weights(self, fetch) -> None:
         self.up, self.down = (Linear(fetch(self.name(n)), fetch(self.name(f"{n}.b")) if self.bias else None) for n in ("up", "down"))
 
+    in_two_pieces = True
+
+    def begin(self, ctx: StepContext, x):
+        return self.up.squared_relu(x)
+
+    def finish(self, ctx: StepContext, x, begun, stream: ResidualStream):
+        return self.down.add_or_defer(begun, stream)
+
     def forward(self, ctx: StepContext, x, stream: ResidualStream):
-        return self.down.add_or_defer(self.up.squared_relu(x), stream)
+        return self.finish(ctx, x, self.begin(ctx, x), stream)
 
 
 class MixtureOfExperts(FeedForward):
@@ -193,12 +201,20 @@ class MixtureOfExperts(FeedForward):
     def _combine(self, into, y, sel, weights, x, assign: bool = False) -> None:
         grouped_ops.moe_combine(into, y, sel, weights, assign=assign, x=x if self.identity else None, experts=self.experts)
 
-    def forward(self, ctx: StepContext, x, stream: ResidualStream):
-        y, sel, weights = self._routed(ctx, x)
+    in_two_pieces = True
+
+    def begin(self, ctx: StepContext, x):
+        return self._routed(ctx, x)
+
+    def finish(self, ctx: StepContext, x, begun, stream: ResidualStream):
+        y, sel, weights = begun
         if self.shared_size:
             self.shared_down.add_into(self._shared_act(x), stream.residual_after_flush(), None)
         self._combine(stream.residual_after_flush(), y, sel, weights, x)
         return None
+
+    def forward(self, ctx: StepContext, x, stream: ResidualStream):
+        return self.finish(ctx, x, self.begin(ctx, x), stream)
 
     def output_terms(self, ctx: StepContext, x):
         y, sel, weights = self._routed(ctx, x)

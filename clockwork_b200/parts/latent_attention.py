@@ -71,6 +71,10 @@ class LatentAttention(Mixer):
     def cache_need(self) -> PagedKVNeed:
         return PagedKVNeed(1, self.kv_rank + self.rot, None, planes=1)
 
+    def reserve_for_steps(self, max_seqs: int, max_ctx: int) -> None:
+        if self.device.type == "cuda" and self.dtype == torch.bfloat16:
+            latent_ops.reserve_scratch(self.device, self.kv_rank, self.rot)
+
     def tensor_decls(self):
         h, heads = self.hidden_size, self.heads
         if self.q_rank is not None:

@@ -2,7 +2,8 @@
 
 ``parallel_residual``: a single norm feeds both, ``n = norm(h); h += mixer(n) + ffn(n)``.
 ``parallel_residual_two_norms``: each has a norm of its own, ``h += mixer(norm1(h)) + ffn(norm2(h))``; one kernel makes both
-norms in one pass over the rows.
+norms in one pass over the rows, and what of the feed-forward does not touch the residual (``FeedForward.begin``) runs on a
+second stream beside the mixer, joined before its last product (or the experts' weighted sum) adds into the residual.
 
 Tensor prefixes: ``<layer>.norm1`` (and ``<layer>.norm2``), ``<layer>.mix``, ``<layer>.mlp``.  A layer without a feed-forward
 names the kind ``none`` (and has no second norm).  The sublayers' output
@@ -12,10 +13,14 @@ products add into the float32 residual in their epilogues, the mixer first, so t
 
 from __future__ import annotations
 
+import torch
+
 from ..config.model_spec import LayerSpec
+from ..ops.library import serial_launch
 from ..weights.decl import TensorDecl
 from .base import Block, Norm, ResidualStream, StepContext
 from .registry import build_part, register_block
+from .side_by_side import side_stream
 
 
 class ParallelResidualBlock(Block):
@@ -79,6 +84,8 @@ class NormPair(Norm):
 
 
 class TwoNormParallelBlock(ParallelResidualBlock):
+    concurrent = True  # the feed-forward on a second stream beside the mixer
+
     def __init__(self, layer: LayerSpec, dtype, device) -> None:
         super().__init__(layer, dtype, device)
         if self.ffn is not None:
@@ -87,6 +94,7 @@ class TwoNormParallelBlock(ParallelResidualBlock):
                 if not hasattr(norm, "forward_with"):
                     raise ValueError(f"norm kind {norm.spec.kind!r} cannot share a pass with another")
             self.norm = NormPair(self.norm, second)
+        self._forked = self._joined = None  # events of the fork and the join (made at first use)
 
     def tensor_decls(self):
         yield from super().tensor_decls()
@@ -99,9 +107,26 @@ class TwoNormParallelBlock(ParallelResidualBlock):
             return
         x, y = self.norm.forward(stream, ctx.status)
         stream.next_norm = None
+        if not (self.concurrent and y.is_cuda and self.ffn.in_two_pieces):
+            stream.push(self.mixer.forward(ctx, x, view, stream))
+            stream.next_norm = following_norm
+            stream.push(self.ffn.forward(ctx, y, stream))
+            stream.next_norm = None
+            return
+        if self._forked is None:
+            self._forked, self._joined = torch.cuda.Event(), torch.cuda.Event()
+        main, side = torch.cuda.current_stream(y.device), side_stream(y.device)
+        self._forked.record(main)
+        side.wait_event(self._forked)  # the norms are ready (and everything the step's stream did before)
+        with torch.cuda.stream(side):
+            begun = self.ffn.begin(ctx, y)
+            self._joined.record(side)
         stream.push(self.mixer.forward(ctx, x, view, stream))
+        stream.flush()
+        main.wait_event(self._joined)
         stream.next_norm = following_norm
-        stream.push(self.ffn.forward(ctx, y, stream))
+        with serial_launch():  # (what reads the second stream's results starts when both streams have got here)
+            stream.push(self.ffn.finish(ctx, y, begun, stream))
         stream.next_norm = None
 
 

@@ -31,7 +31,7 @@ from .registry import build_part, register_mixer
 _side_streams: dict[int, "torch.cuda.Stream"] = {}  # one second stream per device, shared by every layer
 
 
-def _side_stream(device: torch.device) -> "torch.cuda.Stream":
+def side_stream(device: torch.device) -> "torch.cuda.Stream":
     index = device.index if device.index is not None else torch.cuda.current_device()
     stream = _side_streams.get(index)
     if stream is None:
@@ -119,7 +119,7 @@ class SideBySide(Mixer):
         if self.concurrent and x.is_cuda:
             if self._forked is None:
                 self._forked, self._joined = torch.cuda.Event(), torch.cuda.Event()
-            main, side = torch.cuda.current_stream(x.device), _side_stream(x.device)
+            main, side = torch.cuda.current_stream(x.device), side_stream(x.device)
             self._forked.record(main)
             side.wait_event(self._forked)  # x is ready (and everything the step's stream did before)
             with torch.cuda.stream(side):

@@ -691,6 +691,38 @@ def test_a_gate_per_head_in_the_per_head_product(heads, n, k, dtype):
         grouped_ops.per_head_product(a.to(DEV, dtype), k, w.to(DEV, dtype), out, n, head_gate=gate.to(DEV)[:, : heads - 1])
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", ["A", "C", "D"])
+def test_the_feed_forward_on_a_second_stream_changes_nothing(name, dtype, dirs):
+    """The feed-forward's kernels run on a second stream beside the mixer's: the same bits as one after the other, in
+    prompts, portions and captured single-token steps."""
+    from clockwork_b200.parts.parallel_block import TwoNormParallelBlock
+
+    tokens = tokens_for(CONFIGS[name][0], 120, salt=15)
+    results = []
+    for concurrent in (True, False):
+        TwoNormParallelBlock.concurrent = concurrent
+        try:
+            run = Replay(dirs[name], name, dtype, 256)
+            for portion in cut(tokens, [70, 3, 17, 1, 1, 1, 1, 1, 25]):
+                run.step({"a": portion})
+            results.append(run.of("a"))
+        finally:
+            TwoNormParallelBlock.concurrent = True
+    assert torch.equal(results[0], results[1])
+
+
+def test_how_the_keys_of_a_latent_are_cut():
+    """Few rows over a long context are cut until the blocks fill the GPU, short contexts and long portions are not; the
+    scratch holds every plan."""
+    for tokens, seqs, heads, portion, context, want in (
+            (1, 1, 16, 1, 4096, (True, 64)), (8, 8, 16, 1, 4096, (True, 18)), (8, 8, 16, 1, 60, (True, 1)), (64, 64, 20, 1, 9000, (True, 1)),
+            (2048, 1, 16, 2048, 2048, (False, 1)), (64, 1, 16, 64, 16384, (False, 8)), (3, 1, 8, 2, 5000, (True, 49))):
+        few, parts = latent_ops.plan_parts(tokens, seqs, heads, portion, context)
+        assert (few, parts) == want, (tokens, seqs, heads, portion, context)
+        assert parts == 1 or tokens * heads * parts <= latent_ops.FILL_BLOCKS * latent_ops.TILE_ROWS[1]
+
+
 def test_products_take_the_new_epilogue_only_where_it_belongs():
     x, w = torch.zeros((4, 16), device=DEV), torch.zeros((8, 16), device=DEV)
     assert gemm_ops.linear_relu2(x, w, None).shape == (4, 8)
